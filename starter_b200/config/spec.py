@@ -67,12 +67,34 @@ class InterleavedRopeSpec:
 
 
 @dataclass(frozen=True)
+class LinearRopeScaling:
+    """Every frequency of a rotation divided by ``factor``."""
+
+    factor: float
+
+
+@dataclass(frozen=True)
+class YarnRopeScaling:
+    """Frequencies stretched by parts (YaRN).  With ``d(t) = dims * ln(original / (2 pi t)) / (2 ln base)``, ``lo =
+    max(floor(d(fast)), 0)``, ``hi = min(ceil(d(slow)), dims - 1)``: frequency ``i`` is divided by ``factor`` in the
+    share ``clamp((i - lo) / max(hi - lo, 0.001), 0, 1)`` and kept in the rest; cos and sin are multiplied by
+    ``0.1 ln(factor) + 1``."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
 class PartialRopeSpec:
     """Rotary positions that turn entry ``i`` with entry ``i + dims / 2`` of the first ``dims`` entries of a
-    vector by the angle ``position * base ** (-2i / dims)``; entries from ``dims`` on pass unchanged."""
+    vector by the angle ``position * base ** (-2i / dims)``; entries from ``dims`` on pass unchanged.  ``scaling``: None
+    or how the frequencies are changed (``LinearRopeScaling``, ``YarnRopeScaling``)."""
 
     dims: int
     base: float
+    scaling: Optional[object] = None
     kind: str = "rope_partial"
 
 
@@ -149,9 +171,18 @@ class SinkAttentionSpec:
     Keys have ``head_dim`` entries, values ``value_dim``.
 
     ``fixed_sink`` (a number; needs ``sink`` false): the extra term is ``exp(fixed_sink)`` for every head and the
-    layer has no sink tensor.  ``position`` (an ``InterleavedRopeSpec``): queries and keys are turned by their
-    positions before they are scored.  ``values_from_keys``: the layer has no value projection; a key/value head's
-    value is its key as projected, before any rotation (``value_dim`` = ``head_dim``)."""
+    layer has no sink tensor.  ``position`` (an ``InterleavedRopeSpec`` or a ``PartialRopeSpec``): queries and keys are
+    turned by their positions before they are scored.  ``values_from_keys``: the layer has no value projection; a
+    key/value head's value is its key as projected, before any rotation (``value_dim`` = ``head_dim``).
+
+    Further, for layers without head gates: ``keep_first`` (with ``window``): the sequence's first that many keys stay
+    visible however far behind they are, at their true positions.  ``softcap``: a scaled score ``s`` becomes ``softcap *
+    tanh(s / softcap)`` before the softmax.  ``bias``: q, k and v have biases, added in the projection.  ``conv``: a
+    causal convolution of that many taps over time on every channel of q, k and v, directly behind the projection (its
+    last ``conv - 1`` inputs are per-sequence state).  ``row_norm``: queries and keys are RMS-normed over their whole
+    projections (all heads at once) with plain gains, before the rotation; ``unit_values``: each head's value is
+    divided by its root mean square; both with ``norm_eps``.  ``own_kv`` false: no key and value tensors; the layer
+    reads the cache entry another layer fills (the run order says which) with its own queries."""
 
     hidden_size: int
     num_heads: int
@@ -167,6 +198,14 @@ class SinkAttentionSpec:
     position: Optional[object] = None
     fixed_sink: Optional[float] = None
     values_from_keys: bool = False
+    keep_first: int = 0
+    softcap: Optional[float] = None
+    bias: bool = False
+    conv: Optional[int] = None
+    row_norm: bool = False
+    unit_values: bool = False
+    norm_eps: float = 0.0
+    own_kv: bool = True
     kind: str = "sink_attention"
 
 
@@ -273,14 +312,33 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class ForgetWriteSpec:
+    """A linear recurrence with a ``head_dim x value_dim`` state per head whose forget gate also decides what is written
+    (HGRN2).  ``q = silu(W_q h)``, ``v = W_v h``; per key channel ``f = l + (1 - l) * sigmoid(W_f h + b)`` with a stored
+    lower bound ``l``; ``S <- diag(f) S + (1 - f) v^T``, ``o = S^T q``; each head's ``o`` is RMS-normed with a gain of
+    ``value_dim`` entries shared by the heads, then the output projection."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    value_dim: int
+    norm_eps: float
+    kind: str = "forget_write"
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
-    """Two mixers side by side that read the same input: the result is half the sum of their outputs, each first
-    RMS-normed over the model width with a plain gain of its own."""
+    """Two mixers side by side that read the same input.  ``join`` ``"norm_mean"``: the result is half the sum of their
+    outputs, each first RMS-normed over the model width with a plain gain of its own; ``"scaled_sum"``: ``left_scale *
+    left + right_scale * right``."""
 
     hidden_size: int
     left: object
     right: object
-    norm_eps: float
+    norm_eps: float = 0.0
+    join: str = "norm_mean"
+    left_scale: float = 1.0
+    right_scale: float = 1.0
     kind: str = "parallel"
 
     @property
@@ -308,7 +366,7 @@ class RoutedExpertsSpec:
 
     ``scoring`` ``"softmax_top"``: the weights are the softmax over the chosen logits alone;
     ``"sigmoid_normalised"``: the chosen experts' ``sigmoid(logit)`` divided by their sum (+ 1e-20), times
-    ``weight_scale``.  ``expert`` ``"gated_clamped"``: ``down(g * sigmoid(1.702 g) * (u + 1))`` with ``g =
+    ``weight_scale``; ``"sigmoid"``: the plain ``sigmoid(logit)`` times ``weight_scale``.  ``expert`` ``"gated_clamped"``: ``down(g * sigmoid(1.702 g) * (u + 1))`` with ``g =
     min(gate(x), limit)``, ``u = clamp(up(x), -limit, limit)``; ``"relu2"``: ``down(relu(up(x))^2)``, no gate
     and no limit; ``"gated_silu"``: ``down(silu(gate(x)) * up(x))``, no limit.
 
@@ -320,7 +378,10 @@ class RoutedExpertsSpec:
     ``identity_experts``: the router has that many outputs more than there are experts; one of those, chosen,
     stands for an expert that hands its input on (times its weight) and has no tensors.  Groups are formed over
     experts and identity experts together.  ``shared_size`` > 0: a gated expert of that inner size (``"gated_silu"``
-    form) runs for every token and is added times ``sigmoid(sg . x)``, one learnt vector."""
+    form) runs for every token and is added times ``sigmoid(sg . x)``, one learnt vector.
+
+    ``weigh_input``: a chosen expert's weight multiplies its input instead of its output (``expert(w * x)``; not for
+    ``"gated_clamped"`` experts, identity experts or a shared expert)."""
 
     hidden_size: int
     intermediate_size: int
@@ -336,6 +397,7 @@ class RoutedExpertsSpec:
     group_keep: int = 1
     identity_experts: int = 0
     shared_size: int = 0
+    weigh_input: bool = False
     kind: str = "routed_experts"
 
 
@@ -365,9 +427,11 @@ class DepthAverageSpec:
 @dataclass(frozen=True)
 class HyperConnectionSpec:
     """How one sublayer reads from and writes to ``streams`` residual streams: ``in`` and ``out``
-    vectors of that length and a ``[from, to]`` mixing matrix."""
+    vectors of that length and a ``[from, to]`` mixing matrix.  ``channel_scale`` (the model width): the sublayer's
+    output is multiplied by a learnt vector of that size before it is written (None: it is not)."""
 
     streams: int
+    channel_scale: Optional[int] = None
     kind: str = "hyper"
 
 

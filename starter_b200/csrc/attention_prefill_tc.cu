@@ -28,14 +28,19 @@
 // attention_sink.cu): the penalty r1 log2(1 + r2 (p - j)) is taken off a score as it leaves tensor
 // memory (S is unscaled there, so the penalty is divided by the scale first); a row masks the keys
 // before its own chunk; the sink is the state a row's softmax starts from (reference = sink log2(e),
-// sum = 1); the gate multiplies the row's result.  The queries may lie at the front of wider rows
-// (a stacked projection): the tensor map of Q covers those rows.
+// sum = 1); the gate multiplies the row's result; scores may be capped (softcap.cuh); a window may keep the
+// sequence's first keys visible, whose pages then come in front of the window's in the walk.  The queries may
+// lie at the front of wider rows (a stacked projection): the tensor map of Q covers those rows.
+// Keys and values have sizes of their own there, up to 128 each, in shared-memory tiles of one or two 64-entry
+// chunks: S runs over the keys' real entries; V's entries behind the real ones arrive as the zeros TMA fills in,
+// and the output columns they give are not stored.
 //
 // Every wait on an mbarrier gives up after WAIT_LIMIT_NS, raises bit 16 of *status and lets the
 // block drain its copies, free its tensor memory and return.
 #include <cuda.h>
 
 #include "common.cuh"
+#include "softcap.cuh"
 #include "tensor_map.cuh"
 
 #define TC_BQ 128
@@ -212,16 +217,20 @@ __device__ __forceinline__ uint32_t instr_desc(int n, int b_mn_major) {
 }
 
 // What the EXT instance takes besides: r1, r2 (float [heads], both or neither), sink (float [heads] or null),
-// gate (float [tokens, heads] or null), chunk (0: none).
+// gate (float [tokens, heads] or null), chunk (0: none), keep (the first keys a window or chunk keeps visible), the
+// cap of the scores as scale / cap and cap / scale (S is scaled after it; 0: none), the entries of a key and a value.
 struct TcExtras {
   const float* r1;
   const float* r2;
   const float* sink;
   const float* gate;
   int chunk;
+  int keep;
+  float cap_in, cap_out;
+  int dim, vdim;
 };
 
-template <int D, bool EXT>
+template <int DC, int VC, bool EXT>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -231,10 +240,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ tile_seq, const int* __restrict__ tile_first,
                             int heads, int kv_heads, float scale_log2, int window, int* status, int list_of_blocks,
                             TcExtras ex) {
-  constexpr int DC = D / 64;                        // 64-element (128-byte) chunks of the head
+  // DC, VC: 64-element (128-byte) chunks of a key and of a value
+  const int dim = EXT ? ex.dim : DC * 64, vdim = EXT ? ex.vdim : VC * 64;
   constexpr int SUB = 128 * 128;                    // bytes of a [128 rows x 128 bytes] sub-tile
   constexpr int Q_BYTES = DC * SUB;                 // one tile of 128 queries
-  constexpr int KV_BYTES = DC * SUB;                // keys (or values) of 128 tokens
+  constexpr int KV_BYTES = (DC > VC ? DC : VC) * SUB;   // room for the keys (or values) of 128 tokens
   constexpr int P_BYTES = 2 * SUB;                  // [128 queries x 128 keys] bfloat16
   constexpr uint32_t TMEM_COLS = 512;               // S of both tiles: 2 x 128; O of both tiles: 2 x 128
   extern __shared__ uint8_t smem_raw[];
@@ -265,10 +275,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
   if (window > 0 && pos0 - window + 1 > 0) lo = pos0 - window + 1;
   if (EXT && ex.chunk > 0 && pos0 / ex.chunk * ex.chunk > lo) lo = pos0 / ex.chunk * ex.chunk;
   const int page_lo = lo / SB_PAGE_TOKENS, page_hi = hi / SB_PAGE_TOKENS;
-  // steps of two pages (128 keys) that each tile of 128 queries needs, counted from page_lo
+  // the walk's pages: those of kept keys in front of page_lo, then page_lo and on
+  const int kept = EXT && ex.keep > 0 ? min((ex.keep + SB_PAGE_TOKENS - 1) / SB_PAGE_TOKENS, page_lo) : 0;
+  auto page_of = [&](int n) { return EXT && n < kept ? n : page_lo + n - kept; };
+  // steps of two pages (128 keys) that each tile of 128 queries needs
   int n_tile[2];
-  n_tile[0] = ((pos0 + min(rows_valid, TC_BQ) - 1) / SB_PAGE_TOKENS - page_lo) / 2 + 1;
-  n_tile[1] = rows_valid > TC_BQ ? (page_hi - page_lo) / 2 + 1 : 0;
+  n_tile[0] = ((pos0 + min(rows_valid, TC_BQ) - 1) / SB_PAGE_TOKENS - page_lo + kept) / 2 + 1;
+  n_tile[1] = rows_valid > TC_BQ ? (page_hi - page_lo + kept) / 2 + 1 : 0;
   const int n_steps = max(n_tile[0], n_tile[1]);
 
   if (threadIdx.x == 0) {
@@ -304,18 +317,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       if (elected) mbar_expect_tx(&q_full, q_tiles * Q_BYTES);
       for (int t = 0; t < q_tiles; ++t)
         for (int c = 0; c < DC; ++c)
-          if (elected) tma_load_2d(q_sm + t * Q_BYTES + c * SUB, &map_q, &q_full, head * D + c * 64, q_row0 + t * TC_BQ);
+          if (elected) tma_load_2d(q_sm + t * Q_BYTES + c * SUB, &map_q, &q_full, head * dim + c * 64, q_row0 + t * TC_BQ);
       // Keys alternate between buffers 0 and 1 and run a step ahead of the values, which have
       // buffer 2: K0 V0 K1 | K2 V1 | K3 V2 ...  (S of step i+1 is issued early in step i, PV late.)
       auto load = [&](bool is_v, int i) -> bool {
         const int b = is_v ? 2 : (i & 1), use = is_v ? i : (i >> 1);
         if (use > 0 && !__all_sync(0xffffffffu, mbar_wait(&empty[b], (use - 1) & 1, abort))) return false;
-        if (elected) mbar_expect_tx(&full[b], KV_BYTES);
+        const int chunks = is_v ? VC : DC;
+        if (elected) mbar_expect_tx(&full[b], chunks * SUB);
         const bool withheld = is_v && i == *(volatile int*)&tc_withhold_step;   // tests only
         for (int half = 0; half < (withheld ? 1 : 2); ++half) {
-          const int page = pages[min(page_lo + 2 * i + half, page_hi)];
+          const int page = pages[min(page_of(2 * i + half), page_hi)];
           const int row = (page * kv_heads + kvh) * SB_PAGE_TOKENS;
-          for (int c = 0; c < DC; ++c)
+          for (int c = 0; c < chunks; ++c)
             if (elected) tma_load_2d(ring + b * KV_BYTES + c * SUB + half * 8192, is_v ? &map_v : &map_k, &full[b], c * 64, row);
         }
         return true;
@@ -343,13 +357,14 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (n_mine > 0) {
       // the whole warp waits and computes descriptors; one elected lane issues (see the producer)
       const bool elected = elect_one();
-      const uint32_t idesc_s = instr_desc(TC_BK, 0), idesc_o = instr_desc(D, 1);
+      const uint32_t idesc_s = instr_desc(TC_BK, 0), idesc_o = instr_desc((vdim + 15) & ~15, 1);
       const uint32_t q_addr = smem_u32(q_sm + t * Q_BYTES), p_addr = smem_u32(p_sm + t * P_BYTES);
       // S = Q K^T: k runs over the head in steps of 16 (32 bytes inside a 128-byte chunk)
       auto issue_s = [&](int buf) {
         if (elected) {
 #pragma unroll
-          for (int k = 0; k < D / 16; ++k) {
+          for (int k = 0; k < DC * 4; ++k) {
+            if (EXT && k * 16 >= dim) break;
             const uint32_t off = (k >> 2) * SUB + (k & 3) * 32;
             umma_bf16(tmem_base + t * TC_BK, smem_desc(q_addr + off, 16),
                       smem_desc(smem_u32(ring + buf * KV_BYTES) + off, 16), idesc_s, k > 0 ? 1u : 0u);
@@ -446,9 +461,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       ok = mbar_wait(&s_ready[t], i & 1, abort);
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-      const int j0 = (page_lo + 2 * i) * SB_PAGE_TOKENS;
-      const bool edge = j0 + TC_BK - 1 > pos0 + t * TC_BQ ||
-                        (window > 0 && j0 <= pos0 + t * TC_BQ + TC_BQ - window) || (EXT && j0 < tile_lo);
+      // the first keys of the step's two pages (neighbours, but for the step between the kept pages and the others)
+      const int jp[2] = {page_of(2 * i) * SB_PAGE_TOKENS, page_of(2 * i + 1) * SB_PAGE_TOKENS};
+      const bool edge = jp[1] + SB_PAGE_TOKENS - 1 > pos0 + t * TC_BQ ||
+                        (window > 0 && jp[0] <= pos0 + t * TC_BQ + TC_BQ - window) || (EXT && jp[0] < tile_lo);
       float sv[64];
       uint32_t pk[32];
       float mx = -INFINITY, rs = 0.f, rs_hi = 0.f;   // the row sum in two halves (packed adds)
@@ -456,8 +472,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       // half h of the row of S from tensor memory, masked where the step touches an edge
       auto load_half = [&](int h) {
         tmem_load64(tmem_s + h * 64, sv);
+        const int j0 = h ? jp[1] : jp[0];
+        if (EXT && ex.cap_out > 0.f) {
+#pragma unroll
+          for (int e = 0; e < 64; ++e) sv[e] = ex.cap_out * tanh_fast(sv[e] * ex.cap_in);
+        }
         if (EXT && ex.r1) {
-          const float far = (float)(pos - j0 - h * 64);       // the distance to this half's first key
+          const float far = (float)(pos - j0);                // the distance to this half's first key
 #pragma unroll
           for (int e = 0; e < 64; ++e)
             sv[e] -= pen1 * __log2f(fmaf(pen2, fmaxf(far - (float)e, 0.f), 1.f));
@@ -465,8 +486,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         if (edge) {
 #pragma unroll
           for (int e = 0; e < 64; ++e) {
-            const int j = j0 + h * 64 + e;
-            if (j > pos || (window > 0 && j <= pos - window) || (EXT && j < row_lo)) sv[e] = -INFINITY;
+            const int j = j0 + e;
+            if (j > pos || (((window > 0 && j <= pos - window) || (EXT && j < row_lo)) && !(EXT && j < ex.keep))) sv[e] = -INFINITY;
           }
         }
       };
@@ -525,7 +546,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
           if (!ok) break;
           asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
 #pragma unroll 1
-          for (int c = 0; c < D; c += 32) {
+          for (int c = 0; c < vdim; c += 32) {
             float ov[32];
             tmem_load32(tmem_o + c, ov);
 #pragma unroll
@@ -567,14 +588,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       float inv = 1.f / l_run;
       if (EXT && ex.gate && valid)
         inv *= ex.gate[((size_t)seq_q_start[seq] + q_first + t * TC_BQ + r) * heads + head];
-      bf16* dst = out + ((size_t)seq_q_start[seq] + q_first + t * TC_BQ + r) * ((size_t)heads * D) + (size_t)head * D;
+      bf16* dst = out + ((size_t)seq_q_start[seq] + q_first + t * TC_BQ + r) * ((size_t)heads * vdim) + (size_t)head * vdim;
 #pragma unroll 1
-      for (int c = 0; c < D; c += 32) {
+      for (int c = 0; c < vdim; c += 32) {
         float ov[32];
         tmem_load32(tmem_o + c, ov);
         if (valid) {
 #pragma unroll
           for (int d = 0; d < 32; d += 8) {
+            if (EXT && c + d >= vdim) break;
             uint32_t w[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
@@ -600,21 +622,20 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 
 // ------------------------------------------------------------------------------------------ host
 
-template <int D, bool EXT>
+template <int DC, int VC, bool EXT>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out,
                   const int* block_table, int table_stride, const int* seq_slot, const int* seq_q_start,
                   const int* seq_q_len, const int* seq_kv_len, const int* tile_seq, const int* tile_first,
                   int n_tiles, int heads, int kv_heads, float scale, int window, int* status, int list_of_blocks,
-                  cudaStream_t s, TcExtras ex = TcExtras{nullptr, nullptr, nullptr, nullptr, 0}) {
-  constexpr int DC = D / 64;
-  const int smem = (2 * DC + 4 + TC_RING * DC) * 128 * 128 + 1024;
+                  cudaStream_t s, TcExtras ex = TcExtras{nullptr, nullptr, nullptr, nullptr, 0, 0, 0.f, 0.f, DC * 64, VC * 64}) {
+  const int smem = (2 * DC + 4 + TC_RING * (DC > VC ? DC : VC)) * 128 * 128 + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<DC, VC, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  return launch_dependent(attention_prefill_tc_kernel<D, EXT>, dim3(heads, n_tiles), dim3(TC_THREADS), smem, s, mq, mk,
+  return launch_dependent(attention_prefill_tc_kernel<DC, VC, EXT>, dim3(heads, n_tiles), dim3(TC_THREADS), smem, s, mq, mk,
                           mv, (bf16*)out, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len,
                           tile_seq, tile_first, heads, kv_heads, scale * 1.4426950408889634f, window, status,
                           list_of_blocks, ex);
@@ -663,7 +684,7 @@ int sb_attention_prefill_tc(const void* q, void* out, const void* k_store, const
     cudaMemcpyToSymbolAsync(tc_wait_limit_ns, &next_limit_ns, sizeof(next_limit_ns), 0, cudaMemcpyHostToDevice, s);
     cudaStreamSynchronize(s);
   }
-  rc = head_dim == 64 ? launch<64, false>(ARGS) : launch<128, false>(ARGS);
+  rc = head_dim == 64 ? launch<1, 1, false>(ARGS) : launch<2, 2, false>(ARGS);
   if (test_run) {
     cudaStreamSynchronize(s);
     next_withhold_step = -1;
@@ -677,33 +698,35 @@ int sb_attention_prefill_tc(const void* q, void* out, const void* k_store, const
 }
 
 // The same for attention with a distance penalty, chunks, a sink and head gates (see attention_sink.cu): q
-// points at rows of q_width entries (a multiple of 8) whose first heads * head_dim are the queries; out is
-// [n_tokens, heads * head_dim]; keys and values both have head_dim entries (64 or 128); scale > 0.
+// points at rows of q_width entries (a multiple of 8) whose first heads * dim are the queries; out is
+// [n_tokens, heads * vdim]; dim is a multiple of 16 and vdim of 8, both 16 to 128; scale > 0.  keep: the first keys a
+// window or chunk keeps visible; cap: the scores' cap; 0: none.
 int sb_sink_attention_tcgen05(const void* q, int q_width, void* out, const void* k_store, const void* v_store,
                               const int* block_table, int table_stride, const int* seq_slot, const int* seq_q_start,
                               const int* seq_q_len, const int* seq_kv_len, const int* tile_seq, const int* tile_first,
-                              int n_tiles, int n_tokens, int n_pages, int heads, int kv_heads, int head_dim, float scale,
+                              int n_tiles, int n_tokens, int n_pages, int heads, int kv_heads, int dim, int vdim, float scale,
                               const float* r1, const float* r2, const float* sink, const float* gate, int chunk, int window,
-                              int* status, int list_of_blocks, cudaStream_t s) {
+                              int keep, float cap, int* status, int list_of_blocks, cudaStream_t s) {
   if (n_tiles == 0) return 0;
-  if (kv_heads <= 0 || heads % kv_heads || !(scale > 0.f)) return -2;
-  if (head_dim != 64 && head_dim != 128) return -2;
-  if ((r1 == nullptr) != (r2 == nullptr) || q_width % 8 || q_width < heads * head_dim) return -2;
+  if (kv_heads <= 0 || heads % kv_heads || !(scale > 0.f) || keep < 0) return -2;
+  if (dim < 16 || dim > 128 || dim % 16 || vdim < 16 || vdim > 128 || vdim % 8) return -2;
+  if ((r1 == nullptr) != (r2 == nullptr) || q_width % 8 || q_width < heads * dim) return -2;
   if (((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_store | (uintptr_t)v_store) & 15) return -2;
   CUtensorMap mq, mk, mv;
   int rc = sb_make_map(&mq, q, n_tokens, q_width, TC_BQ);
   if (rc) return rc;
   const long long kv_rows = (long long)n_pages * kv_heads * SB_PAGE_TOKENS;
-  rc = sb_make_map(&mk, k_store, kv_rows, head_dim, SB_PAGE_TOKENS);
+  rc = sb_make_map(&mk, k_store, kv_rows, dim, SB_PAGE_TOKENS);
   if (rc) return rc;
-  rc = sb_make_map(&mv, v_store, kv_rows, head_dim, SB_PAGE_TOKENS);
+  rc = sb_make_map(&mv, v_store, kv_rows, vdim, SB_PAGE_TOKENS);
   if (rc) return rc;
-  const TcExtras ex{r1, r2, sink, gate, chunk > 0 ? chunk : 0};
-  if (head_dim == 64)
-    return launch<64, true>(mq, mk, mv, out, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len,
-                            tile_seq, tile_first, n_tiles, heads, kv_heads, scale, window, status, list_of_blocks, s, ex);
-  return launch<128, true>(mq, mk, mv, out, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len,
-                           tile_seq, tile_first, n_tiles, heads, kv_heads, scale, window, status, list_of_blocks, s, ex);
+  const TcExtras ex{r1, r2, sink, gate, chunk > 0 ? chunk : 0, chunk > 0 || window > 0 ? keep : 0,
+                    cap > 0.f ? scale / cap : 0.f, cap > 0.f ? cap / scale : 0.f, dim, vdim};
+#define ARGS mq, mk, mv, out, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len, tile_seq, \
+             tile_first, n_tiles, heads, kv_heads, scale, window, status, list_of_blocks, s, ex
+  if (dim <= 64) return vdim <= 64 ? launch<1, 1, true>(ARGS) : launch<1, 2, true>(ARGS);
+  return vdim <= 64 ? launch<2, 1, true>(ARGS) : launch<2, 2, true>(ARGS);
+#undef ARGS
 }
 
 }  // extern "C"

@@ -7,7 +7,10 @@
 //   softmax:      the denominator holds one more term exp(sink_h): a key that has no value
 //   head output:  times gate[i, h], a number per token and head that arrives as sigmoid(g_h . x_i)
 //
-// Each of the four (penalty, chunk, sink, gate) is switched by its pointer or size, so a design may use
+//   kept keys:    with a window, the keys j < keep stay visible however far behind they are
+//   capped:       a scaled score s becomes cap * tanh(s / cap)
+//
+// Each of these (penalty, chunk, sink, gate, kept keys, cap) is switched by its pointer or size, so a design may use
 // any of them alone.  Keys have `dim` entries, values `vdim`.  Scores, the penalty with its logarithm,
 // the running maximum and sum, the accumulator and the gate are float.
 //
@@ -135,6 +138,148 @@ __global__ void sink_prepare_rot_kernel(T* __restrict__ proj, int proj_width, co
     }
 }
 
+// V consecutive entries as floats and back (V * sizeof(T) == 16: one access; V == 1: any address).
+template <typename T, int V> __device__ __forceinline__ void sink_load(const T* p, float* f) {
+  if (V == 1) {
+    f[0] = to_f<T>(p[0]);
+  } else {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] = to_f<T>(e[i]);
+  }
+}
+template <typename T, int V> __device__ __forceinline__ void sink_store(T* p, const float* f) {
+  if (V == 1) {
+    p[0] = from_f<T>(f[0]);
+  } else {
+    uint4 raw;
+    T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+    for (int i = 0; i < V; ++i) e[i] = from_f<T>(f[i]);
+    *reinterpret_cast<uint4*>(p) = raw;
+  }
+}
+
+// The same for a layer whose queries and keys may be RMS-normed over their whole projections (q_gain, k_gain: float
+// [heads * dim] and [kv_heads * dim], or both null), whose first `rot` entries of a head turn half-split (entry i with
+// entry i + rot / 2; float tables of rot / 2 columns), and whose values may be divided by their root mean square per
+// head (unit_v).  A block a token: the rows' sums of squares, then a piece of V entries a thread (with its partner of
+// the other half where it turns), queries in place, keys into the cache; a warp a value head.
+template <typename T, int V>
+__global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, const int* __restrict__ tok_pos,
+                                         const int* __restrict__ tok_slot, const int* __restrict__ block_table,
+                                         int table_stride, T* __restrict__ k_store, T* __restrict__ v_store,
+                                         const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
+                                         const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
+                                         int unit_v, int heads, int kv_heads, int dim, int vdim, int write) {
+  __shared__ float scratch[33];
+  pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
+  SB_BEHIND_WAIT(proj);
+  SB_BEHIND_WAIT(tok_pos);
+  SB_BEHIND_WAIT(tok_slot);
+  SB_BEHIND_WAIT(block_table);
+  const int row = blockIdx.x, tid = threadIdx.x;
+  T* q = proj + (size_t)row * proj_width;
+  T* k = q + (size_t)heads * dim;
+  const T* v = k + (size_t)kv_heads * dim;
+  const int pos = tok_pos[row], half = rot / 2, pieces = dim / V;
+  const float* cr = cos_t + (size_t)pos * half;
+  const float* sr = sin_t + (size_t)pos * half;
+  auto inverse_rms = [&](const T* x, int n) {
+    float sq = 0.f, f[V];
+    for (int c = tid * V; c < n; c += blockDim.x * V) {
+      sink_load<T, V>(x + c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) sq += f[i] * f[i];
+    }
+    return 1.f / sqrtf(block_sum(sq, scratch) / (float)n + eps);
+  };
+  // piece c of a head: normed, turned with its partner (which this thread handles too) and stored
+  auto turn = [&](const T* from, T* to, const float* gain, float inv, int c) {
+    float x[V], y[V], g[V];
+    const int at = c * V;
+    if (at >= half && at < rot) return;                 // a partner
+    sink_load<T, V>(from + at, x);
+    if (gain) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[i] *= inv * gain[at + i];
+    }
+    if (at >= rot) {
+      sink_store<T, V>(to + at, x);
+      return;
+    }
+    sink_load<T, V>(from + half + at, y);
+    if (gain) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[i] *= inv * gain[half + at + i];
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float co = cr[at + i], si = sr[at + i];
+      g[i] = x[i] * co - y[i] * si;
+      y[i] = y[i] * co + x[i] * si;
+    }
+    sink_store<T, V>(to + at, g);
+    sink_store<T, V>(to + half + at, y);
+  };
+  const float q_inv = q_gain ? inverse_rms(q, heads * dim) : 1.f;
+  const float k_inv = k_gain && write ? inverse_rms(k, kv_heads * dim) : 1.f;
+  for (int e = tid; e < heads * pieces; e += blockDim.x) {
+    const int h = e / pieces, c = e - h * pieces;
+    if (!q_gain && c * V >= half) continue;             // queries in place: nothing to do for entries that stay
+    turn(q + (size_t)h * dim, q + (size_t)h * dim, q_gain ? q_gain + (size_t)h * dim : nullptr, q_inv, c);
+  }
+  if (!write) return;
+  const int page = block_table[(size_t)tok_slot[row] * table_stride + pos / SB_PAGE_TOKENS];
+  const int off = pos % SB_PAGE_TOKENS;
+  for (int e = tid; e < kv_heads * pieces; e += blockDim.x) {
+    const int h = e / pieces, c = e - h * pieces;
+    turn(k + (size_t)h * dim, k_store + page_row(page, h, off, kv_heads, dim), k_gain ? k_gain + (size_t)h * dim : nullptr,
+         k_inv, c);
+  }
+  const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  for (int h = warp; h < kv_heads; h += warps) {
+    const T* from = v + (size_t)h * vdim;
+    T* to = v_store + page_row(page, h, off, kv_heads, vdim);
+    float f[V], inv = 1.f;
+    if (unit_v) {
+      float sq = 0.f;
+      for (int c = lane * V; c < vdim; c += 32 * V) {
+        sink_load<T, V>(from + c, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) sq += f[i] * f[i];
+      }
+      inv = 1.f / sqrtf(warp_sum(sq) / (float)vdim + eps);
+    }
+    for (int c = lane * V; c < vdim; c += 32 * V) {
+      sink_load<T, V>(from + c, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] *= inv;
+      sink_store<T, V>(to + c, f);
+    }
+  }
+}
+
+template <typename T>
+static int sink_prepare_half(void* proj, int proj_width, const int* tok_pos, const int* tok_slot, const int* block_table,
+                             int table_stride, void* k_store, void* v_store, const float* cos_t, const float* sin_t, int rot,
+                             const float* q_gain, const float* k_gain, float eps, int unit_v, int n_tokens, int heads,
+                             int kv_heads, int dim, int vdim, int write, cudaStream_t s) {
+  constexpr int N = 16 / sizeof(T);
+  const bool wide = proj_width % N == 0 && dim % N == 0 && (rot / 2) % N == 0 && vdim % N == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)k_store | (uintptr_t)v_store) & 15) == 0;
+  const int items = heads * dim / (wide ? N : 1);
+  const int threads = items > 512 ? 512 : items > 128 ? 256 : 128;
+#define HALF_GO(V)                                                                                                     \
+  return launch_dependent(sink_prepare_half_kernel<T, V>, dim3(n_tokens), dim3(threads), 0, s, (T*)proj, proj_width,     \
+                          tok_pos, tok_slot, block_table, table_stride, (T*)k_store, (T*)v_store, cos_t, sin_t, rot,    \
+                          q_gain, k_gain, eps, unit_v, heads, kv_heads, dim, vdim, write)
+  if (wide) HALF_GO(N);
+  HALF_GO(1);
+#undef HALF_GO
+}
+
 template <typename T>
 __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out,
                                       const T* __restrict__ k_store, const T* __restrict__ v_store,
@@ -142,7 +287,8 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
                                       const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
                                       const float* __restrict__ r1, const float* __restrict__ r2,
                                       const float* __restrict__ sink, const float* __restrict__ gate, int n_tokens,
-                                      int heads, int kv_heads, int dim, int vdim, float scale, int chunk, int window) {
+                                      int heads, int kv_heads, int dim, int vdim, float scale, int chunk, int window,
+                                      int keep, float cap) {
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(q);
   SB_BEHIND_WAIT(k_store);
@@ -174,7 +320,10 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
   if (chunk > 0) first = pos / chunk * chunk;
   if (window > 0 && pos - window + 1 > first) first = pos - window + 1;
 
-  for (int j0 = first; j0 <= pos; j0 += 4) {
+  // the kept keys in front of the first key of the window (or chunk), then everything from there on
+  for (int part = keep > 0 && first > 0 ? 0 : 1; part < 2; ++part) {
+  const int from = part == 0 ? 0 : first, last = part == 0 ? min(keep, first) - 1 : pos;
+  for (int j0 = from; j0 <= last; j0 += 4) {
     float s[4];
     const T* vrow[4];
 #pragma unroll
@@ -182,7 +331,7 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
       const int j = j0 + u;
       s[u] = 0.f;
       vrow[u] = nullptr;
-      if (j <= pos) {
+      if (j <= last) {
         const int page = pages[j / SB_PAGE_TOKENS];
         const T* kr = k_store + page_row(page, kvh, j % SB_PAGE_TOKENS, kv_heads, dim);
         vrow[u] = v_store + page_row(page, kvh, j % SB_PAGE_TOKENS, kv_heads, vdim);
@@ -197,8 +346,9 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
       s[u] = warp_sum(s[u]) * scale;
+      if (cap > 0.f) s[u] = cap * tanhf(s[u] / cap);
       if (r1) s[u] -= pen1 * log1pf(pen2 * (float)(pos - (j0 + u)));
-      if (j0 + u <= pos) m_new = fmaxf(m_new, s[u]);
+      if (j0 + u <= last) m_new = fmaxf(m_new, s[u]);
     }
     const float alpha = expf(m - m_new);
     l *= alpha;
@@ -206,7 +356,7 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
     for (int i = 0; i < SINK_MAX_D; ++i) acc[i] *= alpha;
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
-      if (j0 + u <= pos) {
+      if (j0 + u <= last) {
         const float p = expf(s[u] - m_new);
         l += p;
 #pragma unroll
@@ -217,6 +367,7 @@ __global__ void sink_attention_kernel(const T* __restrict__ q, int q_stride, T* 
       }
     }
     m = m_new;
+  }
   }
   T* orow = out + ((size_t)token * heads + h) * vdim;
   const float inv = (gate ? gate[(size_t)token * heads + h] : 1.f) / l;
@@ -270,13 +421,30 @@ int sb_sink_prepare_rot(int dtype, void* proj, int proj_width, const int* tok_po
                           heads, kv_heads, dim, vdim, v_from_k, write);
 }
 
+// proj: [n_tokens, proj_width] = [q | k | v] (without `write`: [q]), its queries normed and turned in place; keys and
+// values go to the cache.  q_gain, k_gain: float [heads * dim], [kv_heads * dim], or null (no norm); cos_t, sin_t: float
+// [positions, rot / 2] (unused with rot 0); unit_v: values over their root mean square per head.
+int sb_sink_prepare_half(int dtype, void* proj, int proj_width, const int* tok_pos, const int* tok_slot,
+                         const int* block_table, int table_stride, void* k_store, void* v_store, const float* cos_t,
+                         const float* sin_t, int rot, const float* q_gain, const float* k_gain, float eps, int unit_v,
+                         int n_tokens, int heads, int kv_heads, int dim, int vdim, int write, cudaStream_t s) {
+  if (n_tokens == 0) return 0;
+  if (rot < 0 || rot % 2 || rot > dim || (k_gain && !q_gain)) return -2;
+  if (proj_width < heads * dim + (write ? kv_heads * (dim + vdim) : 0)) return -2;
+#define HALF_ARGS proj, proj_width, tok_pos, tok_slot, block_table, table_stride, k_store, v_store, cos_t, sin_t, rot, q_gain, \
+                  k_gain, eps, unit_v, n_tokens, heads, kv_heads, dim, vdim, write, s
+  return dtype == 0 ? sink_prepare_half<float>(HALF_ARGS) : sink_prepare_half<bf16>(HALF_ARGS);
+#undef HALF_ARGS
+}
+
 // q: rows of q_stride entries whose first heads * dim are the queries; out: [n_tokens, heads * vdim].
 // r1, r2: float [heads] or both null; sink: float [heads] or null; gate: float [n_tokens, heads] or null.
-// chunk, window <= 0: none.
+// chunk, window, keep (the first keys a window keeps), cap <= 0: none.
 int sb_sink_attention(int dtype, const void* q, int q_stride, void* out, const void* k_store, const void* v_store,
                       const int* block_table, int table_stride, const int* tok_slot, const int* tok_pos,
                       const float* r1, const float* r2, const float* sink, const float* gate, int n_tokens, int heads,
-                      int kv_heads, int dim, int vdim, float scale, int chunk, int window, cudaStream_t s) {
+                      int kv_heads, int dim, int vdim, float scale, int chunk, int window, int keep, float cap,
+                      cudaStream_t s) {
   if (dim > 32 * SINK_MAX_D || vdim > 32 * SINK_MAX_D || kv_heads <= 0 || heads % kv_heads) return -2;
   if ((r1 == nullptr) != (r2 == nullptr)) return -2;
   const long long warps = (long long)n_tokens * heads;
@@ -287,11 +455,11 @@ int sb_sink_attention(int dtype, const void* q, int q_stride, void* out, const v
     return launch_dependent(sink_attention_kernel<float>, dim3((unsigned)blocks), dim3(threads), 0, s, (const float*)q,
                             q_stride, (float*)out, (const float*)k_store, (const float*)v_store, block_table,
                             table_stride, tok_slot, tok_pos, r1, r2, sink, gate, n_tokens, heads, kv_heads, dim, vdim,
-                            scale, chunk, window);
+                            scale, chunk, window, keep, cap);
   return launch_dependent(sink_attention_kernel<bf16>, dim3((unsigned)blocks), dim3(threads), 0, s, (const bf16*)q,
                           q_stride, (bf16*)out, (const bf16*)k_store, (const bf16*)v_store, block_table, table_stride,
                           tok_slot, tok_pos, r1, r2, sink, gate, n_tokens, heads, kv_heads, dim, vdim, scale, chunk,
-                          window);
+                          window, keep, cap);
 }
 
 }  // extern "C"

@@ -25,18 +25,28 @@
 // running softmax of its own, and the four (maximum, sum, accumulator) are joined through shared memory
 // at the end.
 //
+// Head sizes that are no instance of the kernel (any multiple of 8 up to 128) run in the next larger one: the tiles'
+// columns from the real size on are filled with zeros by the copies and nothing is stored from them.
+//
+// A window may keep the sequence's first keys visible (`keep`): their pages, as far as they lie in front of the
+// window's first page, are walked before it.  Capped scores: s = cap * log2(e) * tanh(q.k * scale / cap).
+//
 // With n_splits > 1 the pages of a block are dealt out to gridDim.z blocks, which leave (maximum, sum,
 // accumulator) per row in scratch memory for sink_merge_kernel: for steps of few rows (single tokens).
 // The sink belongs to the first part alone.
 #include "common.cuh"
+#include "softcap.cuh"
 
 #define SK_ROWS 64
 #define SK_WARPS 4
 #define SK_THREADS (SK_WARPS * 32)
 
 __device__ __forceinline__ uint32_t sk_smem(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void sk_cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(sk_smem(dst)), "l"(src) : "memory");
+// Entries at .. at + 7 of a row of `n` (16 bytes); zeros when they lie behind its end (n is a multiple of 8).
+__device__ __forceinline__ void sk_cp16(void* dst, const bf16* row, int at, int n) {
+  const int bytes = at < n ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(sk_smem(dst)), "l"(row + (at < n ? at : 0)), "r"(bytes)
+               : "memory");
 }
 __device__ __forceinline__ void sk_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void sk_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
@@ -75,7 +85,8 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                          const int* __restrict__ tile_first, const float* __restrict__ r1,
                          const float* __restrict__ r2, const float* __restrict__ sink,
                          const float* __restrict__ gate, int n_tokens, int heads, int kv_heads, int subs,
-                         int tokens_per_block, float scale_log2, int chunk, int window) {
+                         int tokens_per_block, float scale_log2, int chunk, int window, int dim, int vdim, int keep,
+                         float cap_in, float cap_out) {
   constexpr int CK = D / 8, CV = DV / 8;
   constexpr int K_BYTES = SB_PAGE_TOKENS * D * 2, V_BYTES = SB_PAGE_TOKENS * DV * 2;
   constexpr int KSTEPS = D / 16, NBLK = DV / 8;
@@ -117,26 +128,29 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
   if (chunk > 0) lo = pos0 / chunk * chunk;
   if (window > 0 && pos0 - window + 1 > lo) lo = pos0 - window + 1;
   const int page_lo = lo / SB_PAGE_TOKENS, page_hi = hi / SB_PAGE_TOKENS;
-  const int all_tiles = page_hi - page_lo + 1;
+  // the walk's pages: those of the kept keys that lie in front of page_lo, then page_lo .. page_hi
+  const int kept_pages = keep > 0 ? min((keep + SB_PAGE_TOKENS - 1) / SB_PAGE_TOKENS, page_lo) : 0;
+  const int all_tiles = kept_pages + page_hi - page_lo + 1;
   const int per_split = (all_tiles + n_splits - 1) / n_splits;
   const int t_begin = split * per_split, t_end = min(all_tiles, t_begin + per_split);
   const int n_tiles = max(0, t_end - t_begin);
+  auto page_of = [&](int t) { return t_begin + t < kept_pages ? t_begin + t : page_lo + t_begin + t - kept_pages; };
 
   // ---- stage the queries (rows past the end repeat the last valid row; they are never written)
   for (int idx = tid; idx < SK_ROWS * CK; idx += SK_THREADS) {
     const int r = idx / CK, c = idx % CK;
     const int rr = min(r, rows_valid - 1);
-    const bf16* src = q + (tok0 + rr / group) * (size_t)q_stride + (size_t)(kvh * group + rr % group) * D;
-    sk_cp16(q_tile + sk_offset<D>(r, c), src + c * 8);
+    const bf16* src = q + (tok0 + rr / group) * (size_t)q_stride + (size_t)(kvh * group + rr % group) * dim;
+    sk_cp16(q_tile + sk_offset<D>(r, c), src, c * 8, dim);
   }
   auto load_kv = [&](int t, int buf) {
-    const int page = pages[page_lo + t_begin + t];
-    const bf16* ks = k_store + page_row(page, kvh, 0, kv_heads, D);
-    const bf16* vs = v_store + page_row(page, kvh, 0, kv_heads, DV);
+    const int page = pages[page_of(t)];
+    const bf16* ks = k_store + page_row(page, kvh, 0, kv_heads, dim);
+    const bf16* vs = v_store + page_row(page, kvh, 0, kv_heads, vdim);
     for (int idx = tid; idx < SB_PAGE_TOKENS * CK; idx += SK_THREADS)
-      sk_cp16(k_tiles + buf * K_BYTES + sk_offset<D>(idx / CK, idx % CK), ks + (size_t)idx * 8);
+      sk_cp16(k_tiles + buf * K_BYTES + sk_offset<D>(idx / CK, idx % CK), ks + (size_t)(idx / CK) * dim, idx % CK * 8, dim);
     for (int idx = tid; idx < SB_PAGE_TOKENS * CV; idx += SK_THREADS)
-      sk_cp16(v_tiles + buf * V_BYTES + sk_offset<DV>(idx / CV, idx % CV), vs + (size_t)idx * 8);
+      sk_cp16(v_tiles + buf * V_BYTES + sk_offset<DV>(idx / CV, idx % CV), vs + (size_t)(idx / CV) * vdim, idx % CV * 8, vdim);
   };
   // the penalties of page t: entry [g][x] belongs to the distance pos0 - j0 - 63 + x (negative ones are masked)
   // (thread x forms entry x of every head's table: 128 threads, 128 entries)
@@ -144,7 +158,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
   if (r1) __syncthreads();
   auto make_penalties = [&](int t) {
     if (!r1 || tid >= tokens_valid + 63) return;
-    const float d = (float)max(pos0 - (page_lo + t_begin + t) * SB_PAGE_TOKENS - 63 + tid, 0);
+    const float d = (float)max(pos0 - page_of(t) * SB_PAGE_TOKENS - 63 + tid, 0);
     for (int g = 0; g < group; ++g) pen_tab[g * 128 + tid] = pen_coef[2 * g] * __log2f(fmaf(pen_coef[2 * g + 1], d, 1.f));
   };
   if (n_tiles > 0) load_kv(0, 0);
@@ -197,7 +211,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const int buf = t & 1;
     const uint8_t* kt = k_tiles + buf * K_BYTES;
     const uint8_t* vt = v_tiles + buf * V_BYTES;
-    const int j0 = (page_lo + t_begin + t) * SB_PAGE_TOKENS;
+    const int j0 = page_of(t) * SB_PAGE_TOKENS;
     if (share_keys) {
       // this warp's 16 keys of the page: S (two blocks of 8 keys), softmax, one k-step of P V
       float s2[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
@@ -216,9 +230,9 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         for (int e = 0; e < 4; ++e) {
           const int h = e >> 1;
           const int jj = warp * 16 + nb * 8 + (lane & 3) * 2 + (e & 1);
-          float v = s2[nb][e] * scale_log2;
+          float v = cap_out > 0.f ? cap_out * tanh_fast(s2[nb][e] * cap_in) : s2[nb][e] * scale_log2;
           if (r1) v -= pen_tab[row_pen[h] - jj];
-          if (j0 + jj > row_pos[h] || j0 + jj < row_lo[h]) v = -INFINITY;
+          if (j0 + jj > row_pos[h] || (j0 + jj < row_lo[h] && j0 + jj >= keep)) v = -INFINITY;
           s2[nb][e] = v;
           mx[h] = fmaxf(mx[h], v);
         }
@@ -274,7 +288,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     }
 
     // scale, penalty, mask, online softmax
-    const bool edge = j0 + SB_PAGE_TOKENS - 1 > pos0 || j0 < lo_last;
+    const bool edge = j0 + SB_PAGE_TOKENS - 1 > pos0 || (j0 < lo_last && j0 + SB_PAGE_TOKENS > keep);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int nb = 0; nb < 8; ++nb) {
@@ -282,9 +296,9 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       for (int e = 0; e < 4; ++e) {
         const int h = e >> 1;
         const int jj = nb * 8 + (lane & 3) * 2 + (e & 1);
-        float v = s[nb][e] * scale_log2;
+        float v = cap_out > 0.f ? cap_out * tanh_fast(s[nb][e] * cap_in) : s[nb][e] * scale_log2;
         if (r1) v -= pen_tab[row_pen[h] - jj];
-        if (edge && (j0 + jj > row_pos[h] || j0 + jj < row_lo[h])) v = -INFINITY;
+        if (edge && (j0 + jj > row_pos[h] || (j0 + jj < row_lo[h] && j0 + jj >= keep))) v = -INFINITY;
         s[nb][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -369,6 +383,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const size_t n_rows = (size_t)n_tokens * heads;
     for (int idx = tid; idx < rows_valid * DV; idx += SK_THREADS) {
       const int r = idx / DV, c = idx - r * DV;
+      if (c >= vdim) continue;
       float M = -INFINITY;
 #pragma unroll
       for (int w = 0; w < SK_WARPS; ++w) M = fmaxf(M, meet[(size_t)(w * 16 + r) * LD + DV]);
@@ -382,9 +397,9 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       }
       const size_t grow = (tok0 + r / group) * heads + kvh * group + r % group;
       if (n_splits == 1) {
-        out[grow * DV + c] = from_f<bf16>(a * (gate ? gate[grow] : 1.f) / L);
+        out[grow * vdim + c] = from_f<bf16>(a * (gate ? gate[grow] : 1.f) / L);
       } else {
-        part_acc[((size_t)split * n_rows + grow) * DV + c] = a;
+        part_acc[((size_t)split * n_rows + grow) * vdim + c] = a;
         if (c == 0) {
           part_ml[((size_t)split * n_rows + grow) * 2] = M;
           part_ml[((size_t)split * n_rows + grow) * 2 + 1] = L;
@@ -401,19 +416,19 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const size_t grow = token * heads + row_head[h];
     if (n_splits == 1) {
       const float f = (gate ? gate[grow] : 1.f) / l_run[h];
-      bf16* dst = out + grow * DV;
+      bf16* dst = out + grow * vdim;
 #pragma unroll
       for (int n = 0; n < NBLK; ++n) {
         const int col = n * 8 + (lane & 3) * 2;
-        *reinterpret_cast<uint32_t*>(dst + col) = sk_pack(o[n][2 * h] * f, o[n][2 * h + 1] * f);
+        if (n * 8 < vdim) *reinterpret_cast<uint32_t*>(dst + col) = sk_pack(o[n][2 * h] * f, o[n][2 * h + 1] * f);
       }
     } else {
       const size_t n_rows = (size_t)n_tokens * heads;
-      float* pa = part_acc + ((size_t)split * n_rows + grow) * DV;
+      float* pa = part_acc + ((size_t)split * n_rows + grow) * vdim;
 #pragma unroll
       for (int n = 0; n < NBLK; ++n) {
         const int col = n * 8 + (lane & 3) * 2;
-        *reinterpret_cast<float2*>(pa + col) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+        if (n * 8 < vdim) *reinterpret_cast<float2*>(pa + col) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
       }
       if ((lane & 3) == 0) {
         part_ml[((size_t)split * n_rows + grow) * 2] = m_run[h];
@@ -458,7 +473,7 @@ static int sk_launch(const void* q, int q_stride, void* out, float* part_acc, fl
                      const int* seq_q_start, const int* seq_q_len, const int* seq_kv_len, const int* tile_seq,
                      const int* tile_first, int n_tiles, const float* r1, const float* r2, const float* sink,
                      const float* gate, int n_tokens, int heads, int kv_heads, float scale, int chunk, int window,
-                     int n_splits, int max_q_len, cudaStream_t s) {
+                     int n_splits, int max_q_len, int dim, int vdim, int keep, float cap, cudaStream_t s) {
   const int group = heads / kv_heads;
   const int tokens_per_block = SK_ROWS / group;
   int subs = (SB_PAGE_TOKENS + tokens_per_block - 1) / tokens_per_block;
@@ -474,11 +489,12 @@ static int sk_launch(const void* q, int q_stride, void* out, float* part_acc, fl
                             smem, s, (const bf16*)q, q_stride, (bf16*)out, part_acc, part_ml, (const bf16*)k_store,
                             (const bf16*)v_store, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len,
                             tile_seq, tile_first, r1, r2, sink, gate, n_tokens, heads, kv_heads, subs, tokens_per_block,
-                            scale * 1.4426950408889634f, chunk, window);
+                            scale * 1.4426950408889634f, chunk, window, dim, vdim, window > 0 || chunk > 0 ? keep : 0,
+                            cap > 0.f ? scale / cap : 0.f, cap > 0.f ? cap * 1.4426950408889634f : 0.f);
   if (rc != 0 || n_splits == 1) return rc;
   const int n_rows = n_tokens * heads;
   return launch_dependent(sink_merge_kernel, dim3((n_rows * 32 + 127) / 128), dim3(128), 0, s, (const float*)part_acc,
-                          (const float*)part_ml, gate, (bf16*)out, n_rows, DV, n_splits);
+                          (const float*)part_ml, gate, (bf16*)out, n_rows, vdim, n_splits);
 }
 
 extern "C" {
@@ -486,36 +502,34 @@ extern "C" {
 // q: bfloat16 rows of q_stride entries (a multiple of 8, 16-byte aligned) whose first heads * dim are the
 // queries; out: [n_tokens, heads * vdim].  The seq_* arrays describe the sequences of the step, tile_seq /
 // tile_first its tiles of 64 tokens.  part_acc (float [n_splits, n_tokens * heads, vdim]) and part_ml (float
-// [n_splits, n_tokens * heads, 2]) are scratch for n_splits > 1.  dim and vdim: 16, 32, 64 or 128; up to 64
-// query heads a key/value head.  max_q_len: the most tokens a sequence brings, if known (fewer idle blocks).
+// [n_splits, n_tokens * heads, 2]) are scratch for n_splits > 1.  dim and vdim: multiples of 8 up to 128; up to 64
+// query heads a key/value head.  keep (with a window or chunk): the first keys that stay visible; cap: the scores' cap;
+// 0: none.  max_q_len: the most tokens a sequence brings, if known (fewer idle blocks).
 int sb_sink_attention_tc(const void* q, int q_stride, void* out, float* part_acc, float* part_ml, const void* k_store,
                          const void* v_store, const int* block_table, int table_stride, const int* seq_slot,
                          const int* seq_q_start, const int* seq_q_len, const int* seq_kv_len, const int* tile_seq,
                          const int* tile_first, int n_tiles, const float* r1, const float* r2, const float* sink,
                          const float* gate, int n_tokens, int heads, int kv_heads, int dim, int vdim, float scale,
-                         int chunk, int window, int n_splits, int max_q_len, cudaStream_t s) {
+                         int chunk, int window, int keep, float cap, int n_splits, int max_q_len, cudaStream_t s) {
   if (n_tiles == 0 || n_tokens == 0) return 0;
   if (kv_heads <= 0 || heads % kv_heads || heads / kv_heads > SK_ROWS || n_splits < 1) return -2;
   if ((r1 == nullptr) != (r2 == nullptr) || q_stride % 8 || ((uintptr_t)q % 16)) return -2;
   if (n_splits > 1 && (!part_acc || !part_ml)) return -2;
+  if (dim < 8 || dim % 8 || dim > 128 || vdim < 8 || vdim % 8 || vdim > 128 || keep < 0) return -2;
 #define SK_ARGS q, q_stride, out, part_acc, part_ml, k_store, v_store, block_table, table_stride, seq_slot, seq_q_start, \
                 seq_q_len, seq_kv_len, tile_seq, tile_first, n_tiles, r1, r2, sink, gate, n_tokens, heads, kv_heads,     \
-                scale, chunk, window, n_splits, max_q_len, s
-#define SK_BY_V(DD)                                  \
-  switch (vdim) {                                    \
-    case 16: return sk_launch<DD, 16>(SK_ARGS);      \
-    case 32: return sk_launch<DD, 32>(SK_ARGS);      \
-    case 64: return sk_launch<DD, 64>(SK_ARGS);      \
-    case 128: return sk_launch<DD, 128>(SK_ARGS);    \
-    default: return -2;                              \
+                scale, chunk, window, n_splits, max_q_len, dim, vdim, keep, cap, s
+#define SK_BY_V(DD)                                      \
+  {                                                      \
+    if (vdim <= 16) return sk_launch<DD, 16>(SK_ARGS);   \
+    if (vdim <= 32) return sk_launch<DD, 32>(SK_ARGS);   \
+    if (vdim <= 64) return sk_launch<DD, 64>(SK_ARGS);   \
+    return sk_launch<DD, 128>(SK_ARGS);                  \
   }
-  switch (dim) {
-    case 16: SK_BY_V(16)
-    case 32: SK_BY_V(32)
-    case 64: SK_BY_V(64)
-    case 128: SK_BY_V(128)
-    default: return -2;
-  }
+  if (dim <= 16) SK_BY_V(16)
+  if (dim <= 32) SK_BY_V(32)
+  if (dim <= 64) SK_BY_V(64)
+  SK_BY_V(128)
 #undef SK_BY_V
 #undef SK_ARGS
 }

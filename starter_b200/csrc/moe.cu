@@ -3,13 +3,16 @@
 //
 //   route    z = W_r h + b in float; the `top` largest (the lower index first among equals); their
 //            weights are the softmax over those `top` logits alone (scoring 0), or their sigmoids divided
-//            by the sum of those sigmoids (+ 1e-20) and multiplied by a constant (scoring 1).
+//            by the sum of those sigmoids (+ 1e-20) and multiplied by a constant (scoring 1), or the plain
+//            sigmoids times a constant (scoring 3).
 //   align    the (token, choice) pairs grouped by expert: every expert's pairs fill whole tiles of
 //            rows (32, or 64 for the tensor-core tiles; padded with -1), `tile_expert` names each tile's expert, `n_tiles` counts them.
 //   up       per tile: g = min(gate(h), limit), u = clamp(up(h), -limit, limit),
 //            a = g * sigmoid(1.702 g) * (u + 1), for the tile's rows gathered from h (expert kind 1);
 //            or, for experts without a gate, a = relu(up(h))^2 (expert kind 2); with limit 0 the gated kind
 //            has no clamps and the plain gate: a = silu(gate(h)) * up(h).
+//            A weight that belongs in front of an expert (expert(w h) instead of w expert(h)) multiplies the up
+//            pass's products, which are linear in the row, ahead of the activation; combine then only sums.
 //   down     per tile: the expert's down projection of a, filed at the pair's own place.
 //   combine  out[t] = sum_c weight[t][c] * down[t][c], summed in float in the order of the choices.
 //
@@ -101,10 +104,12 @@ __global__ void moe_route_kernel(const T* __restrict__ h, const float* __restric
     if (lane == 0) {
       float sum = 0.f;
       for (int c = 0; c < top; ++c) {
-        best[c] = scoring == 1 ? 1.f / (1.f + expf(-best[c])) : expf(best[c] - top_max);
+        best[c] = scoring != 0 ? 1.f / (1.f + expf(-best[c])) : expf(best[c] - top_max);
         sum += best[c];
       }
-      if (scoring == 1) {
+      if (scoring == 3) {
+        for (int c = 0; c < top; ++c) weights[(size_t)row * top + c] = best[c] * weight_scale;
+      } else if (scoring == 1) {
         for (int c = 0; c < top; ++c) weights[(size_t)row * top + c] = best[c] / (sum + 1e-20f) * weight_scale;
       } else {
         for (int c = 0; c < top; ++c) weights[(size_t)row * top + c] = best[c] / sum;
@@ -261,7 +266,7 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(256)
 moe_tile_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ y, const int* __restrict__ sorted,
                 const int* __restrict__ tile_expert, const int* __restrict__ n_tiles, int k_dim, int n_out, int top,
-                float limit) {
+                float limit, const float* __restrict__ in_scale) {
   __shared__ float xs[MOE_BM][MOE_BK + 1];
   constexpr bool UP = MODE != 0;
   constexpr int NW = MODE == 1 ? 2 : 1;
@@ -274,6 +279,7 @@ moe_tile_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict_
   SB_BEHIND_WAIT(sorted);
   SB_BEHIND_WAIT(tile_expert);
   SB_BEHIND_WAIT(n_tiles);
+  SB_BEHIND_WAIT(in_scale);
   const int tile = blockIdx.x;
   if (tile >= n_tiles[0]) return;
   const int e = tile_expert[tile];
@@ -327,16 +333,17 @@ moe_tile_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict_
   for (int i = 0; i < 2; ++i) {
     const int m = ty * 2 + i;
     const int pair = src[m];
+    const float by = UP && in_scale && pair >= 0 ? in_scale[pair] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx + 16 * j;
       if (n >= n_out) continue;
       if (MODE == 1) {
-        const float g = rnd<T>(acc[0][i][j]), u = rnd<T>(acc[NW - 1][i][j]);
+        const float g = rnd<T>(acc[0][i][j] * by), u = rnd<T>(acc[NW - 1][i][j] * by);
         const float a = pair >= 0 ? moe_gate(g, u, limit) : 0.f;
         y[((size_t)tile * MOE_BM + m) * n_out + n] = from_f<T>(a);
       } else if (MODE == 2) {
-        const float u = fmaxf(rnd<T>(acc[0][i][j]), 0.f);
+        const float u = fmaxf(rnd<T>(acc[0][i][j] * by), 0.f);
         y[((size_t)tile * MOE_BM + m) * n_out + n] = from_f<T>(pair >= 0 ? u * u : 0.f);
       } else if (pair >= 0) {
         y[(size_t)pair * n_out + n] = from_f<T>(acc[0][i][j]);
@@ -361,7 +368,8 @@ template <int MODE>
 __global__ void __launch_bounds__(256)
 moe_tile_tc_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y,
                    const int* __restrict__ sorted, const int* __restrict__ tile_expert,
-                   const int* __restrict__ n_tiles, int k_dim, int n_out, int top, float limit) {
+                   const int* __restrict__ n_tiles, int k_dim, int n_out, int top, float limit,
+                   const float* __restrict__ in_scale) {
   using namespace nvcuda;
   constexpr bool UP = MODE != 0;
   constexpr int BK = MOE_TC_BK, LD = BK + 8, NW = MODE == 1 ? 2 : 1, STAGES = 3, CLD = MOE_BN + 4;
@@ -381,6 +389,7 @@ moe_tile_tc_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16*
   SB_BEHIND_WAIT(sorted);
   SB_BEHIND_WAIT(tile_expert);
   SB_BEHIND_WAIT(n_tiles);
+  SB_BEHIND_WAIT(in_scale);
   const int tile = blockIdx.x;
   if (tile >= n_tiles[0]) return;
   const int e = tile_expert[tile];
@@ -464,12 +473,13 @@ moe_tile_tc_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16*
     const int n = n0 + nn;
     const int row_pair = src[m];
     if (n >= n_out) continue;
+    const float by = UP && in_scale && row_pair >= 0 ? in_scale[row_pair] : 1.f;
     if (MODE == 1) {
-      const float g = rnd<bf16>(cs[(size_t)m * CLD + nn]), u = rnd<bf16>(cs[((size_t)(NW - 1) * MOE_TC_BM + m) * CLD + nn]);
+      const float g = rnd<bf16>(cs[(size_t)m * CLD + nn] * by), u = rnd<bf16>(cs[((size_t)(NW - 1) * MOE_TC_BM + m) * CLD + nn] * by);
       const float a = row_pair >= 0 ? moe_gate(g, u, limit) : 0.f;
       y[((size_t)tile * MOE_TC_BM + m) * n_out + n] = from_f<bf16>(a);
     } else if (MODE == 2) {
-      const float u = fmaxf(rnd<bf16>(cs[(size_t)m * CLD + nn]), 0.f);
+      const float u = fmaxf(rnd<bf16>(cs[(size_t)m * CLD + nn] * by), 0.f);
       y[((size_t)tile * MOE_TC_BM + m) * n_out + n] = from_f<bf16>(row_pair >= 0 ? u * u : 0.f);
     } else if (row_pair >= 0) {
       y[(size_t)row_pair * n_out + n] = from_f<bf16>(cs[(size_t)m * CLD + nn]);
@@ -499,7 +509,8 @@ template <int MODE>
 __global__ void __launch_bounds__(256)
 moe_tile_big_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y,
                     const int* __restrict__ sorted, const int* __restrict__ tile_expert,
-                    const int* __restrict__ n_tiles, int k_dim, int n_out, int top, float limit) {
+                    const int* __restrict__ n_tiles, int k_dim, int n_out, int top, float limit,
+                    const float* __restrict__ in_scale) {
   constexpr bool UP = MODE != 0;
   // k-slices of 64 (rows of 144 bytes) with one weight block, of 32 (rows of 80 bytes) with two: three stages
   // of either leave room for two blocks an SM
@@ -515,6 +526,7 @@ moe_tile_big_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16
   SB_BEHIND_WAIT(sorted);
   SB_BEHIND_WAIT(tile_expert);
   SB_BEHIND_WAIT(n_tiles);
+  SB_BEHIND_WAIT(in_scale);
   const int tile = blockIdx.x;
   if (tile >= n_tiles[0]) return;
   const int e = tile_expert[tile];
@@ -609,6 +621,7 @@ moe_tile_big_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16
       const int m = wm * 64 + mb * 16 + (lane >> 2) + 8 * h;
       const int row_pair = src[m];
       if (MODE == 0 && row_pair < 0) continue;
+      const float by = UP && in_scale && row_pair >= 0 ? in_scale[row_pair] : 1.f;
       bf16* y_row = y + (MODE == 0 ? (size_t)row_pair : (size_t)tile * MOE_BIG + m) * n_out;
 #pragma unroll
       for (int nb = 0; nb < 4; ++nb) {
@@ -616,12 +629,13 @@ moe_tile_big_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16
         if (n >= n_out) continue;
         float r0, r1;
         if (MODE == 1) {
-          float g0 = rnd<bf16>(acc[0][mb][nb][2 * h]), g1 = rnd<bf16>(acc[0][mb][nb][2 * h + 1]);
-          float u0 = rnd<bf16>(acc[NW - 1][mb][nb][2 * h]), u1 = rnd<bf16>(acc[NW - 1][mb][nb][2 * h + 1]);
+          float g0 = rnd<bf16>(acc[0][mb][nb][2 * h] * by), g1 = rnd<bf16>(acc[0][mb][nb][2 * h + 1] * by);
+          float u0 = rnd<bf16>(acc[NW - 1][mb][nb][2 * h] * by), u1 = rnd<bf16>(acc[NW - 1][mb][nb][2 * h + 1] * by);
           r0 = row_pair >= 0 ? moe_gate(g0, u0, limit) : 0.f;
           r1 = row_pair >= 0 ? moe_gate(g1, u1, limit) : 0.f;
         } else if (MODE == 2) {
-          const float u0 = fmaxf(rnd<bf16>(acc[0][mb][nb][2 * h]), 0.f), u1 = fmaxf(rnd<bf16>(acc[0][mb][nb][2 * h + 1]), 0.f);
+          const float u0 = fmaxf(rnd<bf16>(acc[0][mb][nb][2 * h] * by), 0.f);
+          const float u1 = fmaxf(rnd<bf16>(acc[0][mb][nb][2 * h + 1] * by), 0.f);
           r0 = row_pair >= 0 ? u0 * u0 : 0.f;
           r1 = row_pair >= 0 ? u1 * u1 : 0.f;
         } else {
@@ -652,7 +666,7 @@ template <int MODE>
 __global__ void __launch_bounds__(256)
 moe_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y,
                const int* __restrict__ sorted, const int* __restrict__ tile_expert, const int* __restrict__ n_tiles,
-               int k_dim, int n_out, int top, float limit) {
+               int k_dim, int n_out, int top, float limit, const float* __restrict__ in_scale) {
   constexpr bool UP = MODE != 0;
   constexpr int NW = MODE == 1 ? 2 : 1;
   extern __shared__ __align__(16) float moe_xf[];       // [MOE_FEW][k_dim]
@@ -662,6 +676,7 @@ moe_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __r
   SB_BEHIND_WAIT(sorted);
   SB_BEHIND_WAIT(tile_expert);
   SB_BEHIND_WAIT(n_tiles);
+  SB_BEHIND_WAIT(in_scale);
   const int tile = blockIdx.x;
   if (tile >= n_tiles[0]) return;
   const int e = tile_expert[tile];
@@ -747,10 +762,11 @@ moe_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __r
   static_assert(PER_WARP * MOE_FEW == 32, "a lane for every (weight row, tile row)");
   const int n = n_first + lane / MOE_FEW, r = lane % MOE_FEW;
   if (n < n_out && r < nr) {
+    const float by = UP && in_scale ? in_scale[src[r]] : 1.f;
     if (MODE == 1) {
-      y[((size_t)tile * MOE_FEW + r) * n_out + n] = from_f<bf16>(moe_gate(rnd<bf16>(v0), rnd<bf16>(v1), limit));
+      y[((size_t)tile * MOE_FEW + r) * n_out + n] = from_f<bf16>(moe_gate(rnd<bf16>(v0 * by), rnd<bf16>(v1 * by), limit));
     } else if (MODE == 2) {
-      const float u = fmaxf(rnd<bf16>(v0), 0.f);
+      const float u = fmaxf(rnd<bf16>(v0 * by), 0.f);
       y[((size_t)tile * MOE_FEW + r) * n_out + n] = from_f<bf16>(u * u);
     } else {
       y[(size_t)src[r] * n_out + n] = from_f<bf16>(v0);
@@ -760,22 +776,37 @@ moe_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __r
 
 // The rows of h in the order of `sorted` (a pair's row is h[pair / top]; zeros where a tile is padded), for a
 // product that wants its rows in place: a block a row, 16-byte pieces.  Rows behind the last tile stay unwritten.
+// in_scale (float [pairs] or null) multiplies the rows.
 __global__ void moe_gather_kernel(const bf16* __restrict__ h, const int* __restrict__ sorted,
                                   const int* __restrict__ n_tiles, int tile_rows, int top, bf16* __restrict__ out,
-                                  int width) {
+                                  int width, const float* __restrict__ in_scale) {
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(h);
   SB_BEHIND_WAIT(sorted);
   SB_BEHIND_WAIT(n_tiles);
+  SB_BEHIND_WAIT(in_scale);
   const int row = blockIdx.x;
   if (row >= n_tiles[0] * tile_rows) return;
   const int pair = sorted[row];
   const uint4* from = reinterpret_cast<const uint4*>(h + (size_t)(pair >= 0 ? pair / top : 0) * width);
   uint4* to = reinterpret_cast<uint4*>(out + (size_t)row * width);
+  if (in_scale && pair >= 0) {
+    const float by = in_scale[pair];
+    for (int c = threadIdx.x; c < width / 8; c += blockDim.x) {
+      float f[8];
+      moe_unpack8(from[c], f);
+      uint4 o;
+      __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) e[i] = __floats2bfloat162_rn(f[2 * i] * by, f[2 * i + 1] * by);
+      to[c] = o;
+    }
+    return;
+  }
   for (int c = threadIdx.x; c < width / 8; c += blockDim.x) to[c] = pair >= 0 ? from[c] : make_uint4(0u, 0u, 0u, 0u);
 }
 
-// ids / h (null: every choice is a real expert): a choice from `experts` on stands for the token's own row h[t].
+// weights null: the choices are summed as they are.  ids / h (null: every choice is a real expert): a choice from `experts` on stands for the token's own row h[t].
 // shared / shared_gate (null: none): shared_gate[t] * shared[t] is added.
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ down, const float* __restrict__ weights, T* __restrict__ out,
@@ -794,7 +825,7 @@ __global__ void moe_combine_kernel(const T* __restrict__ down, const float* __re
     float a = 0.f;
     for (int j = 0; j < top; ++j) {
       const bool own = ids && ids[(size_t)row * top + j] >= experts;
-      a += weights[(size_t)row * top + j] *
+      a += (weights ? weights[(size_t)row * top + j] : 1.f) *
            to_f<T>(own ? h[(size_t)row * width + c] : down[((size_t)row * top + j) * width + c]);
     }
     if (shared) a += sg * to_f<T>(shared[(size_t)row * width + c]);
@@ -805,11 +836,12 @@ __global__ void moe_combine_kernel(const T* __restrict__ down, const float* __re
 // up 1: x = h [n_tokens, k_dim], w = [experts, 2 * n_out, k_dim] (gate rows, then up rows), y =
 // [capacity, n_out] in the order of `sorted`, the clamped gated activation.  up 2: the same with w =
 // [experts, n_out, k_dim] and the squared relu.  up 0: x = that y [capacity, k_dim], w = [experts,
-// n_out, k_dim], y = [n_pairs, n_out] by pair.
+// n_out, k_dim], y = [n_pairs, n_out] by pair.  in_scale (up passes): float [n_pairs] that multiplies the products ahead
+// of the activation, or null.
 template <int MODE>
 static int moe_tiles_mode(int dtype, int tile_rows, const void* x, const void* w, void* y, const int* sorted,
                           const int* tile_expert, const int* n_tiles, int max_tiles, int k_dim, int n_out, int top,
-                          float limit, cudaStream_t s) {
+                          float limit, const float* in_scale, cudaStream_t s) {
   if (tile_rows == MOE_FEW) {
     if (dtype != 1 || k_dim % 8 || k_dim > MOE_FEW_MAX_K || ((uintptr_t)x % 16) || ((uintptr_t)w % 16)) return -2;
     const size_t smem = (size_t)MOE_FEW * k_dim * sizeof(float);
@@ -820,7 +852,8 @@ static int moe_tiles_mode(int dtype, int tile_rows, const void* x, const void* w
       configured = smem;
     }
     return launch_dependent(moe_few_kernel<MODE>, dim3(max_tiles, (n_out + MOE_FEW_NB - 1) / MOE_FEW_NB), dim3(256), smem, s,
-                            (const bf16*)x, (const bf16*)w, (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit);
+                            (const bf16*)x, (const bf16*)w, (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit,
+                            in_scale);
   }
   if (tile_rows == MOE_BIG) {
     if (dtype != 1 || k_dim % 16 || n_out % 2 || ((uintptr_t)x % 16) || ((uintptr_t)w % 16) || ((uintptr_t)y % 4)) return -2;
@@ -828,7 +861,8 @@ static int moe_tiles_mode(int dtype, int tile_rows, const void* x, const void* w
     const size_t smem = (size_t)3 * (1 + NW) * MOE_BIG * LD * sizeof(bf16);
     cudaFuncSetAttribute(moe_tile_big_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return launch_dependent(moe_tile_big_kernel<MODE>, dim3(max_tiles, (n_out + MOE_BIG - 1) / MOE_BIG), dim3(256), smem, s,
-                            (const bf16*)x, (const bf16*)w, (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit);
+                            (const bf16*)x, (const bf16*)w, (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit,
+                            in_scale);
   }
   const dim3 grid(max_tiles, (n_out + MOE_BN - 1) / MOE_BN);
   if (tile_rows == MOE_TC_BM) {
@@ -837,14 +871,17 @@ static int moe_tiles_mode(int dtype, int tile_rows, const void* x, const void* w
     const size_t smem = (size_t)3 * (1 + NW) * 64 * (MOE_TC_BK + 8) * sizeof(bf16);
     cudaFuncSetAttribute(moe_tile_tc_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return launch_dependent(moe_tile_tc_kernel<MODE>, grid, dim3(256), smem, s, (const bf16*)x, (const bf16*)w,
-                            (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit);
+                            (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit,
+                            in_scale);
   }
   if (tile_rows != MOE_BM) return -2;
   if (dtype == 0)
     return launch_dependent(moe_tile_kernel<float, MODE>, grid, dim3(256), 0, s, (const float*)x, (const float*)w,
-                            (float*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit);
+                            (float*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit,
+                            in_scale);
   return launch_dependent(moe_tile_kernel<bf16, MODE>, grid, dim3(256), 0, s, (const bf16*)x, (const bf16*)w,
-                          (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit);
+                          (bf16*)y, sorted, tile_expert, n_tiles, k_dim, n_out, top, limit,
+                            in_scale);
 }
 
 extern "C" {
@@ -870,23 +907,24 @@ int sb_moe_tile_rows_for(int dtype, int width, int inner, long long n_pairs, int
 
 // h [.., width] bfloat16 with width a multiple of 8, 16-byte aligned; out [capacity, width].
 int sb_moe_gather(const void* h, const int* sorted, const int* n_tiles, int tile_rows, int top, void* out, int capacity,
-                  int width, cudaStream_t s) {
+                  int width, const float* in_scale, cudaStream_t s) {
   if (capacity == 0) return 0;
   if (width % 8 || ((uintptr_t)h % 16) || ((uintptr_t)out % 16) || top < 1) return -2;
   return launch_dependent(moe_gather_kernel, dim3(capacity), dim3(width / 8 >= 256 ? 256 : 128), 0, s, (const bf16*)h,
-                          sorted, n_tiles, tile_rows, top, (bf16*)out, width);
+                          sorted, n_tiles, tile_rows, top, (bf16*)out, width, in_scale);
 }
 int sb_moe_max_experts() { return MOE_MAX_EXPERTS; }
 int sb_moe_max_top() { return MOE_MAX_TOP; }
 
 // h: [n_tokens, width]; w: float [experts, width]; b: float [experts] or null; ids: int [n_tokens, top];
 // weights: float [n_tokens, top].
-// scoring 0: softmax over the chosen logits; 1: sigmoid scores divided by their sum, times weight_scale.
+// scoring 0: softmax over the chosen logits; 1: sigmoid scores divided by their sum, times weight_scale; 3: plain
+// sigmoid scores times weight_scale.
 int sb_moe_route(int dtype, const void* h, const float* w, const float* b, int* ids, float* weights, int n_tokens,
                  int width, int experts, int top, int scoring, float weight_scale, cudaStream_t s) {
   if (n_tokens == 0) return 0;
   if (experts < 1 || experts > MOE_MAX_EXPERTS || top < 1 || top > MOE_MAX_TOP || top > experts) return -2;
-  if (scoring != 0 && scoring != 1) return -2;
+  if (scoring != 0 && scoring != 1 && scoring != 3) return -2;
   const size_t smem = (size_t)experts * sizeof(float);
   // a step of few rows leaves most SMs idle: a warp an expert (up to 16) shortens the one block a row
   const int threads = n_tokens <= 64 ? (experts >= 16 ? 512 : experts > 4 ? 256 : 128) : 128;
@@ -906,9 +944,9 @@ int sb_moe_align(const int* ids, int n_pairs, int experts, int* sorted, int capa
 
 int sb_moe_tiles(int dtype, int up, int tile_rows, const void* x, const void* w, void* y, const int* sorted,
                  const int* tile_expert, const int* n_tiles, int max_tiles, int k_dim, int n_out, int top, float limit,
-                 cudaStream_t s) {
+                 const float* in_scale, cudaStream_t s) {
   if (max_tiles == 0) return 0;
-#define MOE_ARGS dtype, tile_rows, x, w, y, sorted, tile_expert, n_tiles, max_tiles, k_dim, n_out, top, limit, s
+#define MOE_ARGS dtype, tile_rows, x, w, y, sorted, tile_expert, n_tiles, max_tiles, k_dim, n_out, top, limit, in_scale, s
   if (up == 0) return moe_tiles_mode<0>(MOE_ARGS);
   if (up == 1) return moe_tiles_mode<1>(MOE_ARGS);
   if (up == 2) return moe_tiles_mode<2>(MOE_ARGS);

@@ -1,25 +1,32 @@
 // Linear recurrences with a matrix state S [N x V] per head, over the packed tokens of a step and the
-// per-sequence state in the cache's slots, in two forms that share one kernel:
+// per-sequence state in the cache's slots, in three forms that share one kernel:
 //
 //   state-space (mode 0)   dt = softplus(a_raw + dt_bias), g = exp(-exp(A_log) dt)
 //                          S <- g S + k (dt v)^T,   o = S^T q + D v              (k = B, q = C, v = x)
 //   gated delta (mode 1)   g = exp(-exp(A_log) softplus(a_raw + dt_bias)), beta = sigmoid(b_raw)
 //                          q <- q / sqrt(sum q^2 + 1e-6) * N^-1/2,  k <- k / sqrt(sum k^2 + 1e-6)
 //                          S <- g S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q
+//   forget-write (mode 2)  f = l + (1 - l) sigmoid(z + b) per row of S (z arrives in k's place), q <- silu(q)
+//                          S <- diag(f) S + (1 - f) v^T,   o = S^T q
 //
 // q and k have `G` heads; head h reads head h / (H / G).  S is float in the slot ([H][N][V]), from zero for a
 // new sequence.  Everything but the loads of q, k, v, a_raw, b_raw (working type T) is float; o is stored float.
 //
 // A block owns 32 columns of one head's S for one sequence: 256 threads = 32 columns x 8 lanes; lane p of a
 // column keeps rows p, p + 8, ... (KPT of them) in registers, and the eight lanes of a column sum S^T k and
-// S^T q by shuffles.  (States of more than 64 rows: 16 columns x 16 lanes.)  Both are taken from the state as the token finds it: with u the token's write,
-// (g S + k u^T)^T q = g S^T q + u (k . q), so one round of shuffles a token serves both and the decay is folded
-// into the write.  Tokens arrive in chunks of 16 through two shared-memory buffers (q, k as floats, padded with
-// zeros to 8 * KPT rows; k . q and the unit norms are taken there, a warp a token); the next chunk's global
-// loads are issued before the current chunk is walked and filed after it; outputs leave through shared memory.
+// S^T q by shuffles.  (States of more than 64 rows: 16 columns x 16 lanes.)  Both are taken from the state as the
+// token finds it: with u the token's write, (g S + k u^T)^T q = g S^T q + u (k . q), so one round of shuffles a token
+// serves both and the decay is folded into the write.  In mode 2 the write needs no read-out: S moves by d (v - S)
+// with d = 1 - f = (1 - l) sigmoid(-(z + b)), formed as such (never as one minus a rounded f), and the read-outs of as
+// many tokens as a column has lanes are summed together: each round of shuffles halves the tokens a lane still
+// holds, and lane p ends with token p.
+// Tokens arrive in chunks of 16 through two shared-memory buffers (q, k as floats, padded with zeros to 8 * KPT rows;
+// k . q and the unit norms are taken there, a warp a token); the next chunk's global loads are issued before the
+// current chunk is walked and filed after it; outputs leave through shared memory.
 //
-// Also here: the RMS norm in equal parts of a row with a gate (group_norm_gate), and the mean of two rows each
-// RMS-normed with a gain of its own (norm_pair_mean).
+// Also here: the RMS norm in equal parts of a row with a gate or without (group_norm_gate), and two ways to join two
+// rows: the mean of both, each RMS-normed with a gain of its own (norm_pair_mean), and a sum with two constants
+// (scaled_sum).
 #include "common.cuh"
 
 #define SCAN_CT 16
@@ -55,7 +62,9 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
   typedef ScanBuffer<NP, SCAN_COLS> Buffer;
   extern __shared__ __align__(16) unsigned char scan_smem[];
   Buffer* bufs = reinterpret_cast<Buffer*>(scan_smem);
-  float (*os)[SCAN_COLS] = reinterpret_cast<float (*)[SCAN_COLS]>(scan_smem + 2 * sizeof(Buffer));
+  // (rows of the output tile are padded so that the lanes of a column may file one token each without a conflict)
+  constexpr int OS_LD = SCAN_COLS + 32 / P;
+  float (*os)[OS_LD] = reinterpret_cast<float (*)[OS_LD]>(scan_smem + 2 * sizeof(Buffer));
   // (launch_dependents comes at this kernel's end, not its start: a long prompt keeps its blocks for a while)
   pdl_wait();
   SB_BEHIND_WAIT(q);
@@ -80,7 +89,11 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
     const int i = p + P * r;
     S[r] = (col && i < N) ? sp[(size_t)i * V + j] : 0.f;
   }
-  const float rate = expf(A_log[h]), bias = dt_bias[h], skip = (MODE == 0 && D) ? D[h] : 0.f;
+  // mode 2: A_log holds the lower bounds and dt_bias the biases, [H][N] each; a thread always files the same row of S
+  const int my_row = tid % NP;
+  const float rate = MODE == 2 ? (my_row < N ? 1.f - A_log[(size_t)h * N + my_row] : 0.f) : expf(A_log[h]);
+  const float bias = MODE == 2 ? (my_row < N ? dt_bias[(size_t)h * N + my_row] : 0.f) : dt_bias[h];
+  const float skip = (MODE == 0 && D) ? D[h] : 0.f;
   const float q_mult = MODE == 1 ? rsqrtf((float)N) : 1.f;
 
   // a chunk's loads, held in registers while the chunk before is walked
@@ -102,7 +115,7 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
       const bool have = tt < ct && col0 + c < V;
       rv[n] = have ? v[(size_t)(q_start + t0 + tt) * ldv + (size_t)h * V + col0 + c] : from_f<T>(0.f);
     }
-    if (tid < ct) {
+    if (MODE != 2 && tid < ct) {
       const size_t row = (size_t)(q_start + t0 + tid);
       ra = to_f<T>(a_raw[row * lda + h]);
       if (MODE == 1) rb = to_f<T>(b_raw[row * ldb + h]);
@@ -115,18 +128,20 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
     for (int n = 0; n < QK_PER; ++n) {
       const int e = tid + 256 * n;
       if (e < SCAN_CT * NP) {
-        (&b.q[0][0])[e] = to_f<T>(rq[n]);
-        (&b.k[0][0])[e] = to_f<T>(rk[n]);
+        const float qe = to_f<T>(rq[n]), ke = to_f<T>(rk[n]);
+        (&b.q[0][0])[e] = MODE == 2 ? qe / (1.f + expf(-qe)) : qe;
+        (&b.k[0][0])[e] = MODE == 2 ? rate / (1.f + expf(ke + bias)) : ke;
       }
     }
 #pragma unroll
     for (int n = 0; n < V_PER; ++n) (&b.v[0][0])[tid + 256 * n] = to_f<T>(rv[n]);
-    if (tid < ct) {
+    if (MODE != 2 && tid < ct) {
       const float dt = softplus_f(ra + bias);
       b.dec[tid] = -expm1f(-rate * dt);        // the decay's complement 1 - g: see the walk
       b.fac[tid] = MODE == 0 ? dt : 1.f / (1.f + expf(-rb));
     }
     __syncthreads();
+    if (MODE == 2) return;
     for (int tt = warp; tt < ct; tt += 8) {
       float sq = 0.f, sk = 0.f, dot = 0.f;
       for (int i = lane; i < NP; i += 32) {
@@ -159,7 +174,35 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
     const bool more = t0 + SCAN_CT < q_len;
     if (more) fetch(t0 + SCAN_CT);
     const Buffer& b = bufs[which];
-    for (int tt = 0; tt < ct; ++tt) {
+    for (int tb = 0; MODE == 2 && tb < ct; tb += P) {
+      float part[P];
+#pragma unroll
+      for (int i = 0; i < P; ++i) {
+        part[i] = 0.f;
+        if (tb + i < ct) {
+          const float x = b.v[tb + i][jj];
+          float ra2 = 0.f, rb2 = 0.f;
+#pragma unroll
+          for (int r = 0; r < KPT; ++r) {
+            S[r] = fmaf(b.k[tb + i][p + P * r], x - S[r], S[r]);
+            const float s = S[r] * b.q[tb + i][p + P * r];
+            if (r & 1) rb2 += s; else ra2 += s;
+          }
+          part[i] = ra2 + rb2;
+        }
+      }
+#pragma unroll
+      for (int w = P / 2; w >= 1; w >>= 1) {
+        const bool upper = (p & w) != 0;
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+          const float send = upper ? part[i] : part[i + w], keep = upper ? part[i + w] : part[i];
+          part[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        }
+      }
+      if (tb + p < ct) os[tb + p][jj] = part[0];
+    }
+    for (int tt = 0; MODE != 2 && tt < ct; ++tt) {
       // both read-outs come from the state as the token finds it: with u the token's write,
       // (g S + k u^T)^T q = g S^T q + u (k . q), so one round of shuffles a token serves both
       // (the decay g arrives as d = 1 - g and is applied as S - d * S: a g close to one, rounded to a float,
@@ -208,7 +251,7 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
 
 // ------------------------------------------------------------------------------------------ norm in parts, gated
 // A warp a (token, part).  order 0: y = rms(o * silu(z)) * w (the gate in front of the norm); order 1:
-// y = rms(o) * w * silu(z).  w has `wlen` entries and is read at (column mod wlen): a gain of the whole row,
+// y = rms(o) * w * silu(z); order 2: y = rms(o) * w (no gate, z is not read).  w has `wlen` entries and is read at (column mod wlen): a gain of the whole row,
 // or one of a part's size that every part shares.
 // WIDE: a block a (token, part) instead, for parts of many entries.
 template <typename T, bool WIDE>
@@ -239,8 +282,8 @@ __global__ void group_norm_gate_kernel(const float* __restrict__ o, const T* __r
   const float inv = 1.f / sqrtf(sq / (float)psize + eps);
   T* yrow = y + (size_t)token * parts * psize + (size_t)part * psize;
   for (int c = lane; c < psize; c += step) {
-    const float gz = to_f<T>(zrow[c]);
-    const float silu = gz / (1.f + expf(-gz));
+    const float gz = order == 2 ? 0.f : to_f<T>(zrow[c]);
+    const float silu = order == 2 ? 1.f : gz / (1.f + expf(-gz));
     const float gain = w[(part * psize + c) % wlen];
     yrow[c] = from_f<T>(order == 0 ? orow[c] * silu * inv * gain : orow[c] * inv * gain * silu);
   }
@@ -270,6 +313,39 @@ __global__ void norm_pair_mean_kernel(const T* __restrict__ a, const T* __restri
     orow[c] = from_f<T>(0.5f * (to_f<T>(ar[c]) * ia * wa[c] + to_f<T>(br[c]) * ib * wb[c]));
 }
 
+// out = wa * a + wb * b with two constants; V entries a thread (V = 8 / 4: one 16-byte access; V = 1: any address).
+template <typename T, int V>
+__global__ void scaled_sum_kernel(const T* __restrict__ a, const T* __restrict__ b, T* __restrict__ out, float wa,
+                                  float wb, size_t pieces) {
+  pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
+  SB_BEHIND_WAIT(a);
+  SB_BEHIND_WAIT(b);
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= pieces) return;
+  if (V == 1) {
+    out[i] = from_f<T>(wa * to_f<T>(a[i]) + wb * to_f<T>(b[i]));
+    return;
+  }
+  const uint4 ra = reinterpret_cast<const uint4*>(a)[i], rb = reinterpret_cast<const uint4*>(b)[i];
+  const T *ea = reinterpret_cast<const T*>(&ra), *eb = reinterpret_cast<const T*>(&rb);
+  uint4 ro;
+  T* eo = reinterpret_cast<T*>(&ro);
+#pragma unroll
+  for (int e = 0; e < V; ++e) eo[e] = from_f<T>(wa * to_f<T>(ea[e]) + wb * to_f<T>(eb[e]));
+  reinterpret_cast<uint4*>(out)[i] = ro;
+}
+
+template <typename T>
+static int scaled_sum_launch(const void* a, const void* b, void* out, float wa, float wb, size_t total, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const bool wide = total % V == 0 && (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+  const size_t pieces = wide ? total / V : total;
+  const dim3 grid((unsigned)((pieces + 255) / 256));
+  if (wide)
+    return launch_dependent(scaled_sum_kernel<T, V>, grid, dim3(256), 0, s, (const T*)a, (const T*)b, (T*)out, wa, wb, pieces);
+  return launch_dependent(scaled_sum_kernel<T, 1>, grid, dim3(256), 0, s, (const T*)a, (const T*)b, (T*)out, wa, wb, pieces);
+}
+
 template <typename T, int MODE>
 static int scan_launch(int kpt, int lanes, int n_seqs, cudaStream_t s, const void* q, int ldq, const void* k, int ldk,
                        const void* v, int ldv, const void* a_raw, int lda, const void* b_raw, int ldb, const float* A_log,
@@ -277,7 +353,7 @@ static int scan_launch(int kpt, int lanes, int n_seqs, cudaStream_t s, const voi
                        const int* seq_slot, const int* seq_q_start, const int* seq_q_len, int H, int G, int N, int V) {
 #define SCAN_GO(KPT, P)                                                                                                \
   {                                                                                                                    \
-    const size_t smem = 2 * sizeof(ScanBuffer<P * KPT, 256 / P>) + SCAN_CT * (256 / P) * sizeof(float);                 \
+    const size_t smem = 2 * sizeof(ScanBuffer<P * KPT, 256 / P>) + SCAN_CT * (256 / P + 32 / P) * sizeof(float);        \
     if (smem > 48 * 1024)                                                                                              \
       cudaFuncSetAttribute(state_scan_kernel<T, MODE, KPT, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     const dim3 grid(n_seqs, H, (V + 256 / P - 1) / (256 / P));                                                         \
@@ -303,16 +379,17 @@ extern "C" {
 
 int sb_scan_max_state() { return SCAN_MAX_N; }
 
-// mode 0: state-space; 1: gated delta.  q, k: [n_tokens, ld] with G heads of N entries from the pointer on;
-// v: H heads of V; a_raw (and b_raw in mode 1): H entries; A_log, dt_bias (and D in mode 0, or null): float
-// [H]; state: float, a slot's [H][N][V] starts at the pointer; out: float [n_tokens, H * V].
+// mode 0: state-space; 1: gated delta; 2: forget-write.  q, k: [n_tokens, ld] with G heads of N entries from the
+// pointer on; v: H heads of V; a_raw (and b_raw in mode 1): H entries; A_log, dt_bias (and D in mode 0, or null):
+// float [H].  Mode 2: G == H, k holds the forget gate's logits, A_log the lower bounds and dt_bias the logits' biases
+// (float [H * N] each), a_raw and b_raw are unused. state: float, a slot's [H][N][V] starts at the pointer; out: float [n_tokens, H * V].
 int sb_state_scan(int dtype, int mode, const void* q, int ldq, const void* k, int ldk, const void* v, int ldv,
                   const void* a_raw, int lda, const void* b_raw, int ldb, const float* A_log, const float* dt_bias,
                   const float* D, float* state, long long slot_stride, float* out, const int* seq_slot,
                   const int* seq_q_start, const int* seq_q_len, int n_seqs, int H, int G, int N, int V, cudaStream_t s) {
   if (n_seqs == 0) return 0;
-  if (N < 1 || N > SCAN_MAX_N || V < 1 || H < 1 || G < 1 || H % G || (mode != 0 && mode != 1)) return -2;
-  if (mode == 1 && !b_raw) return -2;
+  if (N < 1 || N > SCAN_MAX_N || V < 1 || H < 1 || G < 1 || H % G || mode < 0 || mode > 2) return -2;
+  if ((mode == 1 && !b_raw) || (mode == 2 && G != H)) return -2;
   // 8 lanes a column and 32 columns a block; for states of more than 64 rows in a step whose blocks would not
   // fill the SMs twice (a prompt of one or two sequences), 16 lanes and 16 columns: half the rows a thread, twice
   // the blocks, a shorter chain of sums a token
@@ -322,17 +399,18 @@ int sb_state_scan(int dtype, int mode, const void* q, int ldq, const void* k, in
   while (lanes * kpt < N) kpt *= 2;
 #define SCAN_ARGS kpt, lanes, n_seqs, s, q, ldq, k, ldk, v, ldv, a_raw, lda, b_raw, ldb, A_log, dt_bias, D, state, slot_stride, out, \
                   seq_slot, seq_q_start, seq_q_len, H, G, N, V
+  if (mode == 2) return dtype == 0 ? scan_launch<float, 2>(SCAN_ARGS) : scan_launch<bf16, 2>(SCAN_ARGS);
   if (dtype == 0) return mode == 0 ? scan_launch<float, 0>(SCAN_ARGS) : scan_launch<float, 1>(SCAN_ARGS);
   return mode == 0 ? scan_launch<bf16, 0>(SCAN_ARGS) : scan_launch<bf16, 1>(SCAN_ARGS);
 #undef SCAN_ARGS
 }
 
 // o: float [n_tokens, parts * psize]; z: [n_tokens, ldz] (working type, the gate's entries from the pointer on);
-// w: float [wlen]; y: [n_tokens, parts * psize].  order 0: gate, then norm; 1: norm, then gate.
+// w: float [wlen]; y: [n_tokens, parts * psize].  order 0: gate, then norm; 1: norm, then gate; 2: no gate (z null).
 int sb_group_norm_gate(int dtype, const float* o, const void* z, int ldz, const float* w, int wlen, void* y, int n_tokens,
                        int parts, int psize, float eps, int order, cudaStream_t s) {
   if (n_tokens == 0) return 0;
-  if (parts < 1 || psize < 1 || wlen < 1 || (order != 0 && order != 1)) return -2;
+  if (parts < 1 || psize < 1 || wlen < 1 || order < 0 || order > 2 || (order != 2 && !z)) return -2;
   const long long warps = (long long)n_tokens * parts;
   if (psize > 256) {
     const dim3 grid((unsigned)warps), block(psize >= 1024 ? 256 : 128);
@@ -359,6 +437,13 @@ int sb_norm_pair_mean(int dtype, const void* a, const void* b, const float* wa, 
                             (const float*)b, wa, wb, (float*)out, width, eps);
   return launch_dependent(norm_pair_mean_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, (const bf16*)a, (const bf16*)b,
                           wa, wb, (bf16*)out, width, eps);
+}
+
+// out = wa * a + wb * b over `total` entries of the working type.
+int sb_scaled_sum(int dtype, const void* a, const void* b, void* out, float wa, float wb, long long total, cudaStream_t s) {
+  if (total <= 0) return 0;
+  return dtype == 0 ? scaled_sum_launch<float>(a, b, out, wa, wb, (size_t)total, s)
+                    : scaled_sum_launch<bf16>(a, b, out, wa, wb, (size_t)total, s);
 }
 
 }  // extern "C"

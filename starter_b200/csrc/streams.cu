@@ -8,13 +8,16 @@
 //     y    = sublayer(norm(u))
 //     x_t <- sum_s mix[s][t] * x_s + out[t] * y      every t from the x before the update
 //
+// (With a layer scale y is multiplied by a vector, channel by channel, before it is written.)
+//
 // The update that closes one sublayer and the read that opens the next touch the same S rows, so
 // they are ONE kernel here (as the residual sum and the norm after it are one kernel in the
 // single-stream models): hyper_step applies the pending update of the previous sublayer in place,
 // forms u for the next one and norms it.  With `rows` it does the same for selected rows without
 // writing back, and with in == null it forms the plain sum of the streams: that closes the model.
 //
-// Dynamic Tanh: y = tanh(alpha * x) * w + b with a scalar alpha; no mean, no variance.
+// Norms of u: Dynamic Tanh, y = tanh(alpha * x) * w + b with a scalar alpha (no mean, no variance: a row may be cut
+// into pieces), or the RMS norm u / sqrt(mean(u^2) + eps) * w (hyper_rms: a block takes a whole row).
 #include "common.cuh"
 
 #define SB_MAX_STREAMS 8
@@ -72,7 +75,8 @@ template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const
 // is cut into pieces of blockDim * V columns (blockIdx.y) and a thread owns V consecutive columns.
 template <typename T, int S, int V>
 __global__ void hyper_step_kernel(float* __restrict__ streams, const T* __restrict__ y,
-                                  const float* __restrict__ y_bias, const float* __restrict__ mix_prev,
+                                  const float* __restrict__ y_bias, const float* __restrict__ y_scale,
+                                  const float* __restrict__ mix_prev,
                                   const float* __restrict__ out_prev, const float* __restrict__ in_next,
                                   int norm_kind, const float* __restrict__ alpha_p,
                                   const float* __restrict__ w, const float* __restrict__ b,
@@ -87,8 +91,9 @@ __global__ void hyper_step_kernel(float* __restrict__ streams, const T* __restri
     inw[i] = in_next ? in_next[i] : 1.f;
   }
   const float alpha = norm_kind == 1 ? alpha_p[0] : 0.f;
-  float wv[V], bv[V], biasv[V];
+  float wv[V], bv[V], biasv[V], scalev[V];
   if (c < hidden) {
+    if (y && y_scale) load_v<float, V>(y_scale + c, scalev);
     if (norm_kind == 1) { load_v<float, V>(w + c, wv); load_v<float, V>(b + c, bv); }
     if (y && y_bias) load_v<float, V>(y_bias + c, biasv);
   }
@@ -109,6 +114,10 @@ __global__ void hyper_step_kernel(float* __restrict__ streams, const T* __restri
     if (y_bias) {
 #pragma unroll
       for (int i = 0; i < V; ++i) yv[i] += biasv[i];
+    }
+    if (y_scale) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) yv[i] *= scalev[i];
     }
     float nx[S][V];
 #pragma unroll
@@ -137,6 +146,90 @@ __global__ void hyper_step_kernel(float* __restrict__ streams, const T* __restri
     u[i] = norm_kind == 1 ? tanhf(alpha * a) * wv[i] + bv[i] : a;
   }
   store_v<T, V>(normed + (size_t)out_row * hidden + c, u);
+}
+
+// The same with an RMS norm of u: a block takes a whole row, whose u waits in shared memory (hidden floats) for
+// the sum of squares.
+template <typename T, int S, int V>
+__global__ void hyper_rms_kernel(float* __restrict__ streams, const T* __restrict__ y, const float* __restrict__ y_bias,
+                                 const float* __restrict__ y_scale, const float* __restrict__ mix_prev,
+                                 const float* __restrict__ out_prev, const float* __restrict__ in_next,
+                                 const float* __restrict__ gain, float eps, T* __restrict__ normed,
+                                 const int* __restrict__ rows, int hidden) {
+  extern __shared__ __align__(16) float u_row[];
+  __shared__ float scratch[33];
+  float mix[S * S], outw[S], inw[S];
+#pragma unroll
+  for (int i = 0; i < S * S; ++i) mix[i] = y ? mix_prev[i] : 0.f;
+#pragma unroll
+  for (int i = 0; i < S; ++i) {
+    outw[i] = y ? out_prev[i] : 0.f;
+    inw[i] = in_next ? in_next[i] : 1.f;
+  }
+  pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
+  SB_BEHIND_WAIT(y);
+  SB_BEHIND_WAIT(rows);
+  const int out_row = blockIdx.x;
+  const int in_row = rows ? rows[out_row] : out_row;
+  float* xr = streams + (size_t)in_row * S * hidden;
+  float sq = 0.f;
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    float x[S][V];
+#pragma unroll
+    for (int s = 0; s < S; ++s) load_v<float, V>(xr + (size_t)s * hidden + c, x[s]);
+    if (y) {
+      float yv[V], extra[V];
+      load_v<T, V>(y + (size_t)in_row * hidden + c, yv);
+      if (y_bias) {
+        load_v<float, V>(y_bias + c, extra);
+#pragma unroll
+        for (int i = 0; i < V; ++i) yv[i] += extra[i];
+      }
+      if (y_scale) {
+        load_v<float, V>(y_scale + c, extra);
+#pragma unroll
+        for (int i = 0; i < V; ++i) yv[i] *= extra[i];
+      }
+      float nx[S][V];
+#pragma unroll
+      for (int t = 0; t < S; ++t) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          float a = 0.f;
+#pragma unroll
+          for (int s = 0; s < S; ++s) a += mix[s * S + t] * x[s][i];
+          nx[t][i] = a + outw[t] * yv[i];
+        }
+      }
+#pragma unroll
+      for (int t = 0; t < S; ++t) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[t][i] = nx[t][i];
+        if (!rows) store_v<float, V>(xr + (size_t)t * hidden + c, nx[t]);
+      }
+    }
+    float u[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      float a = 0.f;
+#pragma unroll
+      for (int s = 0; s < S; ++s) a += inw[s] * x[s][i];
+      u[i] = a;
+      sq += a * a;
+    }
+    store_v<float, V>(u_row + c, u);
+  }
+  sq = block_sum(sq, scratch);
+  const float inv = 1.f / sqrtf(sq / (float)hidden + eps);
+  T* o = normed + (size_t)out_row * hidden;
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    float u[V], g[V];
+    load_v<float, V>(u_row + c, u);          // (what this thread itself stored)
+    load_v<float, V>(gain + c, g);
+#pragma unroll
+    for (int i = 0; i < V; ++i) u[i] = u[i] * inv * g[i];
+    store_v<T, V>(o + c, u);
+  }
 }
 
 // Dynamic Tanh on a single stream of the working type, with the residual sum in front of it as the
@@ -176,14 +269,30 @@ __global__ void add_bias_kernel(T* __restrict__ y, const float* __restrict__ bia
 }
 
 template <typename T, int V>
-static int launch_step_v(int S, float* streams, const void* y, const float* y_bias, const float* mix_prev,
-                         const float* out_prev, const float* in_next, int norm_kind, const float* alpha,
-                         const float* w, const float* b, void* normed, const int* rows, int n_rows, int hidden,
-                         cudaStream_t s) {
+static int launch_step_v(int S, float* streams, const void* y, const float* y_bias, const float* y_scale,
+                         const float* mix_prev, const float* out_prev, const float* in_next, int norm_kind,
+                         const float* alpha, const float* w, const float* b, float eps, void* normed, const int* rows,
+                         int n_rows, int hidden, cudaStream_t s) {
+  if (norm_kind == 2) {
+    const int pieces = (hidden + V - 1) / V;
+    const int threads = pieces >= 1024 ? 512 : pieces > 128 ? 256 : 128;
+    const size_t smem = (size_t)hidden * sizeof(float);
+    if (smem > 51200 * sizeof(float)) return -2;
+#define GO(N) case N: {                                                                                                  \
+      if (smem > 48 * 1024)                                                                                              \
+        cudaFuncSetAttribute(hyper_rms_kernel<T, N, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);         \
+      return launch_dependent(hyper_rms_kernel<T, N, V>, dim3(n_rows), dim3(threads), smem, s, streams, (const T*)y,     \
+                              y_bias, y_scale, mix_prev, out_prev, in_next, w, eps, (T*)normed, rows, hidden); }
+    switch (S) {
+      GO(1) GO(2) GO(3) GO(4) GO(5) GO(6) GO(7) GO(8)
+    }
+#undef GO
+    return -2;
+  }
   const int threads = 128;
   const dim3 grid(n_rows, (hidden + threads * V - 1) / (threads * V));
 #define GO(N) case N: return launch_dependent(hyper_step_kernel<T, N, V>, grid, dim3(threads), 0, s, streams, \
-    (const T*)y, y_bias, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, (T*)normed, rows, hidden)
+    (const T*)y, y_bias, y_scale, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, (T*)normed, rows, hidden)
   switch (S) {
     GO(1); GO(2); GO(3); GO(4); GO(5); GO(6); GO(7); GO(8);
   }
@@ -192,14 +301,15 @@ static int launch_step_v(int S, float* streams, const void* y, const float* y_bi
 }
 
 template <typename T>
-static int launch_step(int S, float* streams, const void* y, const float* y_bias, const float* mix_prev,
-                       const float* out_prev, const float* in_next, int norm_kind, const float* alpha,
-                       const float* w, const float* b, void* normed, const int* rows, int n_rows, int hidden,
-                       cudaStream_t s) {
-  const uintptr_t all = (uintptr_t)streams | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)w | (uintptr_t)b | (uintptr_t)normed;
+static int launch_step(int S, float* streams, const void* y, const float* y_bias, const float* y_scale,
+                       const float* mix_prev, const float* out_prev, const float* in_next, int norm_kind,
+                       const float* alpha, const float* w, const float* b, float eps, void* normed, const int* rows,
+                       int n_rows, int hidden, cudaStream_t s) {
+  const uintptr_t all = (uintptr_t)streams | (uintptr_t)y | (uintptr_t)y_bias | (uintptr_t)y_scale | (uintptr_t)w |
+                        (uintptr_t)b | (uintptr_t)normed;
   if (hidden % 4 == 0 && (all & 15) == 0)
-    return launch_step_v<T, 4>(S, streams, y, y_bias, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, normed, rows, n_rows, hidden, s);
-  return launch_step_v<T, 1>(S, streams, y, y_bias, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, normed, rows, n_rows, hidden, s);
+    return launch_step_v<T, 4>(S, streams, y, y_bias, y_scale, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, eps, normed, rows, n_rows, hidden, s);
+  return launch_step_v<T, 1>(S, streams, y, y_bias, y_scale, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, eps, normed, rows, n_rows, hidden, s);
 }
 
 extern "C" {
@@ -226,18 +336,19 @@ int sb_embed_streams(int dtype, const int* tokens, const void* table, float* out
 }
 
 // streams: float [*, S, hidden].  y (null: no pending update) [*, hidden] of the working type, y_bias
-// null or float [hidden]; mix_prev [S, S] ([from][to]), out_prev [S]; in_next [S] or null (plain sum).
+// null or float [hidden], y_scale likewise (y becomes (y + y_bias) * y_scale); mix_prev [S, S] ([from][to]), out_prev
+// [S]; in_next [S] or null (plain sum).  norm_kind 0: none; 1: Dynamic Tanh (alpha, w, b); 2: RMS norm (gain w, eps).
 // normed: [n_rows, hidden] of the working type.  rows null: every row, updated in place; else only
 // those rows and nothing is written back.
 int sb_hyper_step(int dtype, int n_streams, float* streams, const void* y, const float* y_bias,
-                  const float* mix_prev, const float* out_prev, const float* in_next, int norm_kind,
-                  const float* alpha, const float* w, const float* b, void* normed, const int* rows,
-                  int n_rows, int hidden, cudaStream_t s) {
+                  const float* y_scale, const float* mix_prev, const float* out_prev, const float* in_next,
+                  int norm_kind, const float* alpha, const float* w, const float* b, float eps, void* normed,
+                  const int* rows, int n_rows, int hidden, cudaStream_t s) {
   if (n_rows == 0) return 0;
   if (n_streams < 1 || n_streams > SB_MAX_STREAMS) return -2;
   if (dtype == 0)
-    return launch_step<float>(n_streams, streams, y, y_bias, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, normed, rows, n_rows, hidden, s);
-  return launch_step<bf16>(n_streams, streams, y, y_bias, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, normed, rows, n_rows, hidden, s);
+    return launch_step<float>(n_streams, streams, y, y_bias, y_scale, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, eps, normed, rows, n_rows, hidden, s);
+  return launch_step<bf16>(n_streams, streams, y, y_bias, y_scale, mix_prev, out_prev, in_next, norm_kind, alpha, w, b, eps, normed, rows, n_rows, hidden, s);
 }
 
 int sb_add_bias(int dtype, void* y, const float* bias, int n_rows, int width, cudaStream_t s) {

@@ -789,19 +789,21 @@ def embedding_streams(tokens, table, streams: int, status=None, fence=False):
 def hyper_step(streams, dtype, pending=None, read=None, norm=None, rows=None):
     """One kernel around a sublayer of a model with several residual streams (float32 ``[T, S, H]``).
 
-    ``pending = (y, mix, out, bias)``: the output ``y`` ``[T, H]`` of the sublayer before (``bias``
-    float32 ``[H]`` or None is added to it), which updates the streams, each from the
+    ``pending = (y, mix, out, bias, scale)``: the output ``y`` ``[T, H]`` of the sublayer before (``bias``
+    float32 ``[H]`` or None is added to it, then it is multiplied by ``scale``, float32 ``[H]``, None or left
+    out), which updates the streams, each from the
     values before the update, to ``x_t = sum_s mix[s, t] * x_s + out[t] * y``.  ``read``: float32 ``[S]``, the weights of
     the sum ``u = sum_s read[s] * x_s`` that is returned (None: the plain sum of the streams).
-    ``norm = (alpha, weight, bias)`` makes it ``tanh(alpha * u) * weight + bias`` (Dynamic Tanh); None
-    returns ``u``.  The result is ``[T, H]`` in ``dtype``.  With ``rows`` (int32 ``[R]``) only those rows
+    ``norm = (alpha, weight, bias)`` makes it ``tanh(alpha * u) * weight + bias`` (Dynamic Tanh), ``norm = (gain, eps)``
+    the RMS norm of ``u`` times the float32 ``gain``; None returns ``u``.  The result is ``[T, H]`` in ``dtype``.  With ``rows`` (int32 ``[R]``) only those rows
     are computed, the result is ``[R, H]`` and the streams are left as they were; without, the update
     is written into ``streams``."""
     _need(streams, "streams", torch.float32, 3)
     n_tokens, n_streams, hidden = streams.shape
-    y = mix = out = bias = None
+    y = mix = out = bias = scale = None
     if pending is not None:
-        y, mix, out, bias = pending
+        y, mix, out, bias = pending[:4]
+        scale = pending[4] if len(pending) > 4 else None
         _need(y, "y", dtype, 2)
         if tuple(y.shape) != (n_tokens, hidden):
             raise KernelError(f"y {tuple(y.shape)} does not match streams {tuple(streams.shape)}")
@@ -809,10 +811,17 @@ def hyper_step(streams, dtype, pending=None, read=None, norm=None, rows=None):
         _f32(out, "out", (n_streams,))
         if bias is not None:
             _f32(bias, "bias", (hidden,))
+        if scale is not None:
+            _f32(scale, "scale", (hidden,))
     if read is not None:
         _f32(read, "read", (n_streams,))
     alpha = weight = shift = None
-    if norm is not None:
+    kind, eps = 0, 0.0
+    if norm is not None and len(norm) == 2:
+        kind, (weight, eps) = 2, norm
+        _f32(weight, "norm gain", (hidden,))
+    elif norm is not None:
+        kind = 1
         alpha, weight, shift = norm
         _f32(alpha, "alpha")
         _f32(weight, "norm weight", (hidden,))
@@ -823,11 +832,12 @@ def hyper_step(streams, dtype, pending=None, read=None, norm=None, rows=None):
         n_rows = rows.shape[0]
     normed = torch.empty((n_rows, hidden), dtype=dtype, device=streams.device)
     rc = _lib("streams").sb_hyper_step(
-        _code(dtype), n_streams, _ptr(streams), _ptr(y), _ptr(bias), _ptr(mix), _ptr(out), _ptr(read),
-        int(norm is not None), _ptr(alpha), _ptr(weight), _ptr(shift), _ptr(normed), _ptr(rows), n_rows,
+        _code(dtype), n_streams, _ptr(streams), _ptr(y), _ptr(bias), _ptr(scale), _ptr(mix), _ptr(out), _ptr(read),
+        kind, _ptr(alpha), _ptr(weight), _ptr(shift), ctypes.c_float(eps), _ptr(normed), _ptr(rows), n_rows,
         hidden, _stream())
     if rc == -2:
-        raise KernelError(f"the stream kernels take 1 to {max_streams()} streams, not {n_streams}")
+        raise KernelError(f"the stream kernels take 1 to {max_streams()} streams, not {n_streams} (with an RMS norm: rows "
+                          f"of up to 51,200 entries, not {hidden})")
     _check(rc, "hyper_step")
     return normed
 
@@ -1607,7 +1617,7 @@ def moe_limits():
 
 
 #: how the chosen experts' weights are formed from their logits, and the code the router takes
-MOE_SCORINGS = {"softmax_top": 0, "sigmoid_normalised": 1, "softmax_all": 2}
+MOE_SCORINGS = {"softmax_top": 0, "sigmoid_normalised": 1, "softmax_all": 2, "sigmoid": 3}
 #: the experts the tile kernels know, and the code of their up pass (``gated_silu`` is the gated pass without clamps)
 MOE_EXPERTS = {"gated_clamped": 1, "relu2": 2, "gated_silu": 1}
 
@@ -1615,7 +1625,8 @@ MOE_EXPERTS = {"gated_clamped": 1, "relu2": 2, "gated_silu": 1}
 def moe_route(h, router, router_bias, top, scoring="softmax_top", weight_scale=1.0):
     """``(ids int32 [T, top], weights float32 [T, top])``: the ``top`` largest of ``router @ h + bias``
     (float32 ``[E, W]`` and ``[E]`` or None), and either the softmax over those alone or, with ``scoring``
-    ``"sigmoid_normalised"``, their sigmoids divided by their sum (+ 1e-20) times ``weight_scale``."""
+    ``"sigmoid_normalised"``, their sigmoids divided by their sum (+ 1e-20) times ``weight_scale``, or, with
+    ``"sigmoid"``, their plain sigmoids times ``weight_scale``."""
     if scoring not in MOE_SCORINGS:
         raise KernelError(f"no router scoring {scoring!r} (known: {', '.join(MOE_SCORINGS)})")
     _need(h, "h", None, 2)
@@ -1661,7 +1672,7 @@ def moe_route_all(h, router, correction, top, groups=1, keep=1, weight_scale=1.0
 
 
 def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped", tile_rows=None, status=None,
-                identity=False, shared=None, shared_gate=None):
+                identity=False, shared=None, shared_gate=None, weigh_input=False):
     """The chosen experts of every row and their weighted sum: ``gate_up`` ``[E, 2 * F, W]`` (an expert's
     gate rows, then its up rows), ``down`` ``[E, W, F]``; an expert is ``down(g * sigmoid(1.702 g) * (u +
     1))`` with ``g = min(gate(h), limit)`` and ``u = clamp(up(h), -limit, limit)``.  With ``expert``
@@ -1673,7 +1684,8 @@ def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped
 
     ``expert`` ``"gated_silu"``: ``down(silu(gate(h)) * up(h))``, no clamps.  ``identity``: an id from ``E`` on names
     an expert without weights that hands the row itself on.  ``shared`` ``[T, W]`` with ``shared_gate`` float32
-    ``[T]``: ``shared_gate[t] * shared[t]`` is added to row ``t`` of the result."""
+    ``[T]``: ``shared_gate[t] * shared[t]`` is added to row ``t`` of the result.  ``weigh_input``: a choice's weight
+    multiplies its expert's input instead of its output (``expert(w * h)``; not for clamped or identity experts)."""
     if expert not in MOE_EXPERTS:
         raise KernelError(f"no expert kind {expert!r} (known: {', '.join(MOE_EXPERTS)})")
     up_mode = MOE_EXPERTS[expert]
@@ -1681,6 +1693,9 @@ def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped
         limit = 0.0                       # the gated pass without clamps
     elif up_mode == 1 and not limit > 0.0:
         raise KernelError(f"the clamped gate needs a positive limit, not {limit}")
+    if weigh_input and (identity or limit > 0.0):
+        raise KernelError("weights in front of the experts are for experts without clamps, none of them an identity")
+    in_scale, out_scale = (weights, None) if weigh_input else (None, weights)
     _need(h, "h", None, 2)
     if shared is not None:
         _need(shared, "shared", h.dtype, 2)
@@ -1719,7 +1734,8 @@ def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped
     if bm == 256:
         grouped = _lib("gemm_prompt_tcgen05").sb_gemm_prompt_grouped
         gathered = torch.empty((capacity, width), dtype=h.dtype, device=h.device)
-        rc = lib.sb_moe_gather(_ptr(h), _ptr(sorted_pairs), _ptr(n_tiles), bm, top, _ptr(gathered), capacity, width, _stream())
+        rc = lib.sb_moe_gather(_ptr(h), _ptr(sorted_pairs), _ptr(n_tiles), bm, top, _ptr(gathered), capacity, width,
+                               _ptr(in_scale), _stream())
         _check(rc, "moe_gather")
         rc = grouped(_ptr(gathered), _ptr(gate_up), _ptr(act), capacity, inner, width, experts, _ptr(tile_expert),
                      _ptr(n_tiles), max_tiles, None,
@@ -1730,18 +1746,19 @@ def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped
                      _ptr(n_tiles), max_tiles, _ptr(sorted_pairs), 0, 0, ctypes.c_float(0.0), _ptr(status), _stream())
         _check(rc, "moe_down (grouped tcgen05)")
         out = torch.empty_like(h)
-        rc = lib.sb_moe_combine(_code(h.dtype), _ptr(per_pair), _ptr(weights), _ptr(out), n_tokens, width, top, *extras,
+        rc = lib.sb_moe_combine(_code(h.dtype), _ptr(per_pair), _ptr(out_scale), _ptr(out), n_tokens, width, top, *extras,
                                 _stream())
         _check(rc, "moe_combine")
         return out
     rc = lib.sb_moe_tiles(_code(h.dtype), up_mode, bm, _ptr(h), _ptr(gate_up), _ptr(act), _ptr(sorted_pairs), _ptr(tile_expert),
-                          _ptr(n_tiles), max_tiles, width, inner, top, ctypes.c_float(limit), _stream())
+                          _ptr(n_tiles), max_tiles, width, inner, top, ctypes.c_float(limit), _ptr(in_scale), _stream())
     _check(rc, "moe_up")
     rc = lib.sb_moe_tiles(_code(h.dtype), 0, bm, _ptr(act), _ptr(down), _ptr(per_pair), _ptr(sorted_pairs),
-                          _ptr(tile_expert), _ptr(n_tiles), max_tiles, inner, width, top, ctypes.c_float(limit), _stream())
+                          _ptr(tile_expert), _ptr(n_tiles), max_tiles, inner, width, top, ctypes.c_float(limit), None,
+                          _stream())
     _check(rc, "moe_down")
     out = torch.empty_like(h)
-    rc = lib.sb_moe_combine(_code(h.dtype), _ptr(per_pair), _ptr(weights), _ptr(out), n_tokens, width, top, *extras,
+    rc = lib.sb_moe_combine(_code(h.dtype), _ptr(per_pair), _ptr(out_scale), _ptr(out), n_tokens, width, top, *extras,
                                 _stream())
     _check(rc, "moe_combine")
     return out
@@ -1906,6 +1923,52 @@ def sink_prepare_rot(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block_
     _check(rc, "sink_prepare_rot")
 
 
+def sink_prepare_half(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block_table, k_store, v_store, rotation=None,
+                      row_norm=None, unit_values=False, eps=0.0, write_cache=True):
+    """``sink_prepare_rot`` for half-split rotations, with norms: ``proj`` = ``[q | k | v]`` (``[q]`` with ``write_cache``
+    false; up to 7 unused entries may follow).  ``row_norm = (q_gain, k_gain)`` (float32 ``[heads * dim]``, ``[kv_heads *
+    dim]`` or None when nothing is filed): queries and keys are RMS-normed over their whole rows first.  ``rotation`` (a
+    half-split ``Rotation`` or None): entry ``i`` of its leading dimensions turns with entry ``i + dims / 2``.
+    ``unit_values``: a head's value is divided by its root mean square.  Queries change in place, keys and values are
+    filed in the cache; ``eps`` stands inside every root."""
+    _need(proj, "proj", None, 2)
+    n_tokens = proj.shape[0]
+    want = heads * dim + (kv_heads * (dim + vdim) if write_cache else 0)
+    if not want <= proj.shape[1] < want + 8:
+        raise KernelError(f"proj has width {proj.shape[1]}, expected {want} (and up to 7 entries of padding)")
+    _need(tok_pos, "tok_pos", torch.int32, 1)
+    _need(tok_slot, "tok_slot", torch.int32, 1)
+    _need(block_table, "block_table", torch.int32, 2)
+    rot, cos_table, sin_table = 0, None, None
+    if rotation is not None:
+        rot, cos_table, sin_table = rotation.rotary_dim, rotation.cos, rotation.sin
+        if rotation.layout != "half_split" or rot > dim or rot % 2:
+            raise KernelError(f"this kernel turns up to {dim} leading entries of a head in half-split layout; asked for {rot} "
+                              f"in {rotation.layout!r} layout")
+        _need(cos_table, "cos table", torch.float32, 2)
+        _need(sin_table, "sin table", torch.float32, 2)
+        if cos_table.shape[1] != rot // 2 or tuple(sin_table.shape) != tuple(cos_table.shape):
+            raise KernelError(f"rotation tables {tuple(cos_table.shape)} do not turn {rot} entries")
+    q_gain = k_gain = None
+    if row_norm is not None:
+        q_gain, k_gain = row_norm[0], row_norm[1] if write_cache else None
+        _f32(q_gain, "query gain", (heads * dim,))
+        if write_cache:
+            _f32(k_gain, "key gain", (kv_heads * dim,))
+    if write_cache:
+        _need(k_store, "key pages", proj.dtype, 4)
+        _need(v_store, "value pages", proj.dtype, 4)
+        if tuple(k_store.shape[1:]) != (kv_heads, PAGE_TOKENS, dim) or tuple(v_store.shape[1:]) != (kv_heads, PAGE_TOKENS, vdim):
+            raise KernelError(f"cache pages have shapes {tuple(k_store.shape)} / {tuple(v_store.shape)}, expected "
+                              f"[pages, {kv_heads}, {PAGE_TOKENS}, {dim}] / [.., {vdim}]")
+    rc = _lib("attention_sink").sb_sink_prepare_half(
+        _code(proj.dtype), _ptr(proj), proj.shape[1], _ptr(tok_pos), _ptr(tok_slot), _ptr(block_table),
+        block_table.shape[1], _ptr(k_store if write_cache else None), _ptr(v_store if write_cache else None),
+        _ptr(cos_table), _ptr(sin_table), rot, _ptr(q_gain), _ptr(k_gain), ctypes.c_float(eps), int(unit_values), n_tokens,
+        heads, kv_heads, dim, vdim, int(write_cache), _stream())
+    _check(rc, "sink_prepare_half")
+
+
 def _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, gate):
     _need(q, "q", None, 2)
     if q.shape[1] < heads * dim:
@@ -1927,13 +1990,14 @@ def _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, 
 
 
 def sink_attention(q, k_store, v_store, block_table, tok_slot, tok_pos, heads, kv_heads, dim, vdim, scale,
-                   penalty=None, sink=None, gate=None, chunk=None, window=None):
+                   penalty=None, sink=None, gate=None, chunk=None, window=None, keep_first=0, softcap=None):
     """Attention of every query row over its sequence's cached keys, plain kernel (any sizes up to
     ``sink_max_dim()``, both types).  ``q``: rows whose first ``heads * dim`` entries are the queries (a
     stacked projection may carry more behind them).  ``penalty = (r1, r2)``: ``r1_h ln(1 + r2_h (i - j))`` is
     taken off the scaled scores; ``sink``: one more term ``exp(sink_h)`` in the softmax's denominator;
     ``gate`` float32 ``[T, heads]``: multiplies the head's output; ``chunk``: keys of the query's own chunk of
-    that many positions only; ``window``: the most recent that many keys.  Returns ``[T, heads * vdim]``."""
+    that many positions only; ``window``: the most recent that many keys; ``keep_first``: with either, the sequence's
+    first that many keys too; ``softcap``: a scaled score ``s`` becomes ``softcap * tanh(s / softcap)``.  Returns ``[T, heads * vdim]``."""
     r1, r2 = _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, gate)
     _need(block_table, "block_table", torch.int32, 2)
     _need(tok_slot, "tok_slot", torch.int32, 1)
@@ -1942,35 +2006,38 @@ def sink_attention(q, k_store, v_store, block_table, tok_slot, tok_pos, heads, k
     rc = _lib("attention_sink").sb_sink_attention(
         _code(q.dtype), _ptr(q), q.shape[1], _ptr(out), _ptr(k_store), _ptr(v_store), _ptr(block_table),
         block_table.shape[1], _ptr(tok_slot), _ptr(tok_pos), _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate), q.shape[0],
-        heads, kv_heads, dim, vdim, ctypes.c_float(scale), int(chunk or 0), int(window or 0), _stream())
+        heads, kv_heads, dim, vdim, ctypes.c_float(scale), int(chunk or 0), int(window or 0), int(keep_first),
+        ctypes.c_float(softcap or 0.0), _stream())
     _check(rc, "sink_attention")
     return out
 
 
-SINK_TC_DIMS = (16, 32, 64, 128)
+#: the largest key or value head the tensor-core kernel takes (sizes between its instances of 16, 32, 64 and 128
+#: entries run in the next larger one)
+SINK_TC_MAX_DIM = 128
 
 
 def sink_tc_takes(q, heads, kv_heads, dim, vdim) -> bool:
-    """Whether the tensor-core kernel takes these operands: bfloat16, ``dim`` and ``vdim`` of 16, 32, 64 or
+    """Whether the tensor-core kernel takes these operands: bfloat16, ``dim`` and ``vdim`` multiples of 8 up to
     128, up to 64 query heads a key/value head, query rows that start on 16-byte boundaries."""
-    return (q.dtype == torch.bfloat16 and dim in SINK_TC_DIMS and vdim in SINK_TC_DIMS and heads // kv_heads <= 64
-            and q.shape[1] % 8 == 0 and q.data_ptr() % 16 == 0)
+    return (q.dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= SINK_TC_MAX_DIM
+            and heads // kv_heads <= 64 and q.shape[1] % 8 == 0 and q.data_ptr() % 16 == 0)
 
 
-def sink_splits(rows: int, kv_heads: int, chunk, window, kv_hint: int) -> int:
+def sink_splits(rows: int, kv_heads: int, chunk, window, kv_hint: int, keep_first: int = 0) -> int:
     """Into how many parts the pages of a single-token step are cut: enough blocks for two an SM, no part
     shorter than a page, at most 16."""
     keys = max(kv_hint, 1)
     for bound in (chunk, window):
         if bound:
             keys = min(keys, bound)
-    pages = -(-keys // PAGE_TOKENS) + 1
+    pages = -(-keys // PAGE_TOKENS) + 1 + -(-keep_first // PAGE_TOKENS)
     return max(1, min(16, (2 * 148) // max(1, rows * kv_heads), pages))
 
 
 def sink_attention_tc(q, k_store, v_store, block_table, seq_slot, seq_q_start, seq_q_len, seq_kv_len, tile_seq,
                       tile_first, heads, kv_heads, dim, vdim, scale, penalty=None, sink=None, gate=None, chunk=None,
-                      window=None, n_splits=1, max_q_len=0):
+                      window=None, n_splits=1, max_q_len=0, keep_first=0, softcap=None):
     """``sink_attention`` on tensor cores (bfloat16): a block takes one key/value head and the query heads
     that share it for consecutive tokens of a sequence (up to 64 rows), so a page is fetched once for all
     of them.  The ``seq_*`` arrays describe the sequences of the step, ``tile_seq`` / ``tile_first`` list
@@ -1978,8 +2045,8 @@ def sink_attention_tc(q, k_store, v_store, block_table, seq_slot, seq_q_start, s
     a second kernel joins: for steps of few rows."""
     r1, r2 = _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, gate)
     if not sink_tc_takes(q, heads, kv_heads, dim, vdim):
-        raise KernelError(f"the tensor-core attention takes bfloat16 heads of 16, 32, 64 or 128 entries in rows "
-                          f"that are multiples of 8 wide; got {q.dtype}, {dim} / {vdim}, rows of {q.shape[1]}")
+        raise KernelError(f"the tensor-core attention takes bfloat16 heads of up to {SINK_TC_MAX_DIM} entries, a multiple of "
+                          f"8, in rows that are multiples of 8 wide; got {q.dtype}, {dim} / {vdim}, rows of {q.shape[1]}")
     _need(block_table, "block_table", torch.int32, 2)
     for name, t in (("seq_slot", seq_slot), ("seq_q_start", seq_q_start), ("seq_q_len", seq_q_len),
                     ("seq_kv_len", seq_kv_len), ("tile_seq", tile_seq), ("tile_first", tile_first)):
@@ -1995,29 +2062,33 @@ def sink_attention_tc(q, k_store, v_store, block_table, seq_slot, seq_q_start, s
         _ptr(q), q.shape[1], _ptr(out), _ptr(part_acc), _ptr(part_ml), _ptr(k_store), _ptr(v_store), _ptr(block_table),
         block_table.shape[1], _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(tile_seq),
         _ptr(tile_first), tile_seq.shape[0], _ptr(r1), _ptr(r2), _ptr(sink), _ptr(gate), n_tokens, heads, kv_heads,
-        dim, vdim, ctypes.c_float(scale), int(chunk or 0), int(window or 0), n_splits, int(max_q_len), _stream())
+        dim, vdim, ctypes.c_float(scale), int(chunk or 0), int(window or 0), int(keep_first), ctypes.c_float(softcap or 0.0),
+        n_splits, int(max_q_len), _stream())
     _check(rc, "sink_attention_tc", 2 if n_splits > 1 else 1)
     return out
 
 
 def sink_tcgen05_takes(q, dim, vdim) -> bool:
-    """Whether the tcgen05 prompt kernel takes these operands: bfloat16, keys and values of one size, 64 or
-    128, query rows that are a multiple of 8 wide and start on 16-byte boundaries."""
-    return (q.dtype == torch.bfloat16 and dim == vdim and dim in PREFILL_TC_HEAD_DIMS and q.shape[1] % 8 == 0
-            and q.data_ptr() % 16 == 0)
+    """Whether the tcgen05 prompt kernel takes these operands: bfloat16, keys of 16 to 128 entries (a multiple of 16),
+    values of 16 to 128 (a multiple of 8), query rows that are a multiple of 8 wide and start on 16-byte boundaries."""
+    return (q.dtype == torch.bfloat16 and 16 <= dim <= 128 and dim % 16 == 0 and 16 <= vdim <= 128 and vdim % 8 == 0
+            and q.shape[1] % 8 == 0 and q.data_ptr() % 16 == 0)
 
 
 def sink_attention_tcgen05(q, k_store, v_store, block_table, seq_slot, seq_q_start, seq_q_len, seq_kv_len, tile_seq,
                            tile_first, heads, kv_heads, dim, scale, penalty=None, sink=None, gate=None, chunk=None,
-                           window=None, status=None, blocks=None):
+                           window=None, status=None, blocks=None, vdim=None, keep_first=0, softcap=None):
     """``sink_attention`` for prompts on the tcgen05 kernel of ``attention_prefill`` (256 queries of a head a
-    block, S and O in tensor memory), which takes the penalty, the chunks, the sink and the gate as extras.
+    block, S and O in tensor memory), which takes the penalty, the chunks, the sink, the gate,
+    the kept keys, the cap and values of another size (``vdim``) than the keys as extras.
     ``blocks = (block_seq, block_first)``: the work list in blocks of 256 queries (else the tiles of 64 are
     launched and three of four blocks find nothing to do)."""
-    r1, r2 = _sink_check(q, k_store, v_store, heads, kv_heads, dim, dim, penalty, sink, gate)
-    if not sink_tcgen05_takes(q, dim, dim):
-        raise KernelError(f"the tcgen05 attention takes bfloat16 heads of 64 or 128 entries, keys and values alike, in "
-                          f"rows that are multiples of 8 wide; got {q.dtype}, {dim}, rows of {q.shape[1]}")
+    vdim = dim if vdim is None else vdim
+    r1, r2 = _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, gate)
+    if not sink_tcgen05_takes(q, dim, vdim):
+        raise KernelError(f"the tcgen05 attention takes bfloat16 keys of 16 to 128 entries (a multiple of 16) and values of "
+                          f"16 to 128 (a multiple of 8) in rows that are multiples of 8 wide; got {q.dtype}, {dim} / {vdim}, "
+                          f"rows of {q.shape[1]}")
     if not scale > 0:
         raise KernelError("the tcgen05 attention needs a positive scale")
     _need(block_table, "block_table", torch.int32, 2)
@@ -2029,32 +2100,36 @@ def sink_attention_tcgen05(q, k_store, v_store, block_table, seq_slot, seq_q_sta
         for name, t in (("block_seq", blocks[0]), ("block_first", blocks[1])):
             _need(t, name, torch.int32, 1)
     list_seq, list_first = blocks if own_list else (tile_seq, tile_first)
-    out = torch.empty((q.shape[0], heads * dim), dtype=q.dtype, device=q.device)
+    out = torch.empty((q.shape[0], heads * vdim), dtype=q.dtype, device=q.device)
     rc = _lib("attention_prefill_tc").sb_sink_attention_tcgen05(
         _ptr(q), q.shape[1], _ptr(out), _ptr(k_store), _ptr(v_store), _ptr(block_table), block_table.shape[1],
         _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(list_seq), _ptr(list_first),
-        list_seq.shape[0], q.shape[0], k_store.shape[0], heads, kv_heads, dim, ctypes.c_float(scale), _ptr(r1), _ptr(r2),
-        _ptr(sink), _ptr(gate), int(chunk or 0), int(window or 0), _ptr(status), int(own_list), _stream())
+        list_seq.shape[0], q.shape[0], k_store.shape[0], heads, kv_heads, dim, vdim, ctypes.c_float(scale), _ptr(r1), _ptr(r2),
+        _ptr(sink), _ptr(gate), int(chunk or 0), int(window or 0), int(keep_first), ctypes.c_float(softcap or 0.0),
+        _ptr(status), int(own_list), _stream())
     _check(rc, "sink_attention_tcgen05")
     return out
 
 
 def sink_attention_step(q, k_store, v_store, block_table, ctx, heads, kv_heads, dim, vdim, scale, penalty=None,
-                        sink=None, gate=None, chunk=None, window=None):
+                        sink=None, gate=None, chunk=None, window=None, keep_first=0, softcap=None):
     """``sink_attention`` for the step ``ctx`` describes, on the kernel that fits its shape: for bfloat16 the
-    tcgen05 kernel when a sequence brings more than 128 tokens and keys and values have 64 or 128 entries, the
-    mma.sync kernel for other steps and sizes it takes; the plain kernel otherwise (float32, other sizes)."""
+    tcgen05 kernel when a sequence brings more than 128 tokens and it takes the head sizes, the mma.sync kernel for
+    other steps and sizes it takes; the plain kernel otherwise (float32, other sizes)."""
     if ctx.max_q_len > 128 and scale > 0 and sink_tcgen05_takes(q, dim, vdim):
         return sink_attention_tcgen05(q, k_store, v_store, block_table, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
                                       ctx.seq_kv_len, ctx.tile_seq, ctx.tile_first, heads, kv_heads, dim, scale, penalty,
-                                      sink, gate, chunk, window, ctx.status, (ctx.block_seq, ctx.block_first))
+                                      sink, gate, chunk, window, ctx.status, (ctx.block_seq, ctx.block_first), vdim,
+                                      keep_first, softcap)
     if sink_tc_takes(q, heads, kv_heads, dim, vdim):
-        splits = sink_splits(ctx.n_seqs, kv_heads, chunk, window, ctx.max_kv_len) if ctx.max_q_len == 1 else 1
+        splits = 1
+        if ctx.max_q_len == 1:
+            splits = sink_splits(ctx.n_seqs, kv_heads, chunk, window, ctx.max_kv_len, keep_first)
         return sink_attention_tc(q, k_store, v_store, block_table, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
                                  ctx.seq_kv_len, ctx.tile_seq, ctx.tile_first, heads, kv_heads, dim, vdim, scale,
-                                 penalty, sink, gate, chunk, window, splits, ctx.max_q_len)
+                                 penalty, sink, gate, chunk, window, splits, ctx.max_q_len, keep_first, softcap)
     return sink_attention(q, k_store, v_store, block_table, ctx.tok_slot, ctx.tok_pos, heads, kv_heads, dim, vdim,
-                          scale, penalty, sink, gate, chunk, window)
+                          scale, penalty, sink, gate, chunk, window, keep_first, softcap)
 
 
 def linear_gated_clamped(x, weight, limit, status=None):
@@ -2110,7 +2185,7 @@ def short_conv(x, col, channels, taps, bias, in_bias, state, state_at, seq_slot,
     ``y[t, c] = act(bias[c] + sum_j taps[c, K - 1 - j] * (x[t - j, col + c] + in_bias[c]))``, zeros in front of a
     sequence.  ``x`` ``[T, N]`` (the channels are its columns ``col .. col + channels``); ``taps`` float32
     ``[channels, K]``; ``bias``, ``in_bias`` float32 ``[channels]`` or None; ``activation`` None or ``"silu"``.
-    ``state`` float32 ``[slots, M]``: a slot's last ``K - 1`` inputs (``(K - 1) * channels`` floats from
+    ``state`` float32 ``[slots, M]`` (None with one tap): a slot's last ``K - 1`` inputs (``(K - 1) * channels`` floats from
     ``state_at`` on) stand in front of the tokens it brings and are replaced by the step's last ones.
     ``max_q_len``: the most tokens a sequence brings.  Returns ``[T, channels]`` in the type of ``x``."""
     _need(x, "x", None, 2)
@@ -2122,18 +2197,21 @@ def short_conv(x, col, channels, taps, bias, in_bias, state, state_at, seq_slot,
         _f32(bias, "bias", (channels,))
     if in_bias is not None:
         _f32(in_bias, "in_bias", (channels,))
-    _need(state, "state", torch.float32, 2)
-    if col < 0 or col + channels > x.shape[1] or state_at < 0 or state_at + (k - 1) * channels > state.shape[1]:
+    slot_floats = 0
+    if state is not None:
+        _need(state, "state", torch.float32, 2)
+        slot_floats = state.shape[1]
+    if col < 0 or col + channels > x.shape[1] or state_at < 0 or (k > 1 and state_at + (k - 1) * channels > slot_floats):
         raise KernelError(f"{channels} channels from column {col} of rows of {x.shape[1]}, or {k - 1} rows of them from "
-                          f"float {state_at} of a slot's {state.shape[1]}, do not fit")
+                          f"float {state_at} of a slot's {slot_floats}, do not fit")
     if activation not in (None, "silu"):
         raise KernelError(f"the short convolution applies silu or nothing, not {activation!r}")
     n_seqs = _seq_arrays(seq_slot, seq_q_start, seq_q_len)
     y = torch.empty((x.shape[0], channels), dtype=x.dtype, device=x.device)
     rc = _lib("short_conv").sb_short_conv(
         _code(x.dtype), _at(x, col), x.shape[1], _ptr(taps), _ptr(bias), _ptr(in_bias), _ptr(y), channels,
-        _at(state, state_at), ctypes.c_longlong(state.shape[1]), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len),
-        n_seqs, int(max_q_len), channels, k, 1 if activation == "silu" else 0, _stream())
+        _at(state, state_at) if state is not None else _ptr(None), ctypes.c_longlong(slot_floats), _ptr(seq_slot),
+        _ptr(seq_q_start), _ptr(seq_q_len), n_seqs, int(max_q_len), channels, k, 1 if activation == "silu" else 0, _stream())
     if rc == -2:
         raise KernelError(f"the short convolution takes 1 to {conv_max_taps()} taps, not {k}")
     _check(rc, "short_conv")
@@ -2175,7 +2253,7 @@ def glru_scan(u, gates, r_bias, i_bias, lam, decay_scale, proj, y_col, y_bias, s
 
 # ---------------------------------------------------------------------------------------- recurrences with a matrix state
 
-SCAN_MODES = {"state_space": 0, "gated_delta": 1}
+SCAN_MODES = {"state_space": 0, "gated_delta": 1, "forget_write": 2}
 
 
 def scan_max_state() -> int:
@@ -2193,7 +2271,10 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
     ``"state_space"``: ``dt = softplus(a_raw + dt_bias)``, ``S <- exp(-exp(A_log) dt) S + k (dt v)^T``, ``o = S^T q +
     skip * v`` (``b_raw`` None).  ``"gated_delta"``: q and k made unit vectors (``x / sqrt(sum x^2 + 1e-6)``), q times
     ``n_state ** -0.5``; ``S <- exp(-exp(A_log) softplus(a_raw + dt_bias)) S``, ``u = sigmoid(b_raw) (v - S^T k)``, ``S
-    <- S + k u^T``, ``o = S^T q``.  ``state`` float32 ``[slots, M]``: a slot's ``[heads, n_state, v_dim]`` from
+    <- S + k u^T``, ``o = S^T q``.  ``"forget_write"`` (``groups`` = ``heads``; ``a_raw``, ``b_raw`` None): ``q <- silu(q)``,
+    ``k`` holds the logits of a forget gate ``f = A_log + (1 - A_log) sigmoid(k + dt_bias)`` per row of the state, with
+    lower bounds in ``A_log`` and biases in ``dt_bias`` (float32 ``[heads * n_state]`` each); ``S <- diag(f) S + (1 - f)
+    v^T``, ``o = S^T q``.  ``state`` float32 ``[slots, M]``: a slot's ``[heads, n_state, v_dim]`` from
     ``state_at`` on, read at the start and written at the end.  Returns float32 ``[T, heads * v_dim]``."""
     if mode not in SCAN_MODES:
         raise KernelError(f"no recurrence {mode!r} (known: {', '.join(SCAN_MODES)})")
@@ -2210,8 +2291,9 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
         if t.shape[0] != n_tokens or col < 0 or col + width > t.shape[1]:
             raise KernelError(f"{name}: {width} columns from {col} of {tuple(t.shape)} do not fit {n_tokens} tokens")
         args += [_at(t, col), t.shape[1]]
-    _f32(A_log, "A_log", (heads,))
-    _f32(dt_bias, "dt_bias", (heads,))
+    per_head = heads * n_state if mode == "forget_write" else heads
+    _f32(A_log, "A_log", (per_head,))
+    _f32(dt_bias, "dt_bias", (per_head,))
     if skip is not None:
         _f32(skip, "skip", (heads,))
     _need(state, "state", torch.float32, 2)
@@ -2233,20 +2315,24 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
 def group_norm_gate(o, z, z_col, weight, parts, eps, gate_first, dtype):
     """The RMS norm of each of the ``parts`` equal parts of a float32 row ``o`` ``[T, N]`` with ``silu`` of the
     gate ``z`` (columns ``z_col .. z_col + N`` of a ``[T, M]`` tensor of ``dtype``): ``gate_first``: ``rms(o *
-    silu(z)) * w``; else ``rms(o) * w * silu(z)``.  ``weight`` float32 of ``N`` entries, or of one part's size when
+    silu(z)) * w``; else ``rms(o) * w * silu(z)``; with ``z`` None ``rms(o) * w``.  ``weight`` float32 of ``N`` entries, or of one part's size when
     the parts share it.  Returns ``[T, N]`` in ``dtype``."""
     _need(o, "o", torch.float32, 2)
     n_tokens, width = o.shape
-    _need(z, "z", dtype, 2)
     _need(weight, "weight", torch.float32, 1)
-    if parts < 1 or width % parts or z.shape[0] != n_tokens or z_col < 0 or z_col + width > z.shape[1]:
-        raise KernelError(f"rows of {width} in {parts} parts with a gate from column {z_col} of {tuple(z.shape)} do not fit")
+    if parts < 1 or width % parts:
+        raise KernelError(f"rows of {width} do not split into {parts} parts")
+    if z is not None:
+        _need(z, "z", dtype, 2)
+        if z.shape[0] != n_tokens or z_col < 0 or z_col + width > z.shape[1]:
+            raise KernelError(f"rows of {width} in {parts} parts with a gate from column {z_col} of {tuple(z.shape)} do not fit")
     if weight.shape[0] not in (width, width // parts):
         raise KernelError(f"a gain of {weight.shape[0]} entries fits neither the row ({width}) nor a part ({width // parts})")
     y = torch.empty((n_tokens, width), dtype=dtype, device=o.device)
-    rc = _lib("state_scan").sb_group_norm_gate(_code(dtype), _ptr(o), _at(z, z_col), z.shape[1], _ptr(weight),
+    gate, gate_width, order = (_ptr(None), 0, 2) if z is None else (_at(z, z_col), z.shape[1], 0 if gate_first else 1)
+    rc = _lib("state_scan").sb_group_norm_gate(_code(dtype), _ptr(o), gate, gate_width, _ptr(weight),
                                                weight.shape[0], _ptr(y), n_tokens, parts, width // parts,
-                                               ctypes.c_float(eps), 0 if gate_first else 1, _stream())
+                                               ctypes.c_float(eps), order, _stream())
     _check(rc, "group_norm_gate")
     return y
 
@@ -2263,4 +2349,17 @@ def norm_pair_mean(a, b, gain_a, gain_b, eps):
     rc = _lib("state_scan").sb_norm_pair_mean(_code(a.dtype), _ptr(a), _ptr(b), _ptr(gain_a), _ptr(gain_b), _ptr(out),
                                               a.shape[0], a.shape[1], ctypes.c_float(eps), _stream())
     _check(rc, "norm_pair_mean")
+    return out
+
+
+def scaled_sum(a, b, weight_a, weight_b):
+    """``weight_a * a + weight_b * b`` for ``a``, ``b`` ``[T, W]`` and two numbers."""
+    _need(a, "a", None, 2)
+    _need(b, "b", a.dtype, 2)
+    if tuple(a.shape) != tuple(b.shape):
+        raise KernelError(f"rows {tuple(a.shape)} and {tuple(b.shape)} differ")
+    out = torch.empty_like(a)
+    rc = _lib("state_scan").sb_scaled_sum(_code(a.dtype), _ptr(a), _ptr(b), _ptr(out), ctypes.c_float(weight_a),
+                                          ctypes.c_float(weight_b), ctypes.c_longlong(a.numel()), _stream())
+    _check(rc, "scaled_sum")
     return out

@@ -45,6 +45,7 @@ ROLES = {
     "stream_weight": Role(0.25, 0.2, always_32bit=True),  # how streams are read, written and mixed
     "gain_offset": Role(0.0, 0.1, always_32bit=True),    # a norm's gain stored around zero (gain - 1)
     "shift": Role(0.5, 0.2, always_32bit=True),          # how much of the previous token a mix takes
+    "floor": Role(0.4, 0.1, always_32bit=True),          # the lower bound of a forget gate
     "matrix32": Role(0.0, 0.02, always_32bit=True),      # a small projection computed in 32-bit (a router)
 }
 

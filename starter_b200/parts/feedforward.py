@@ -114,6 +114,8 @@ class RoutedExperts(Part):
                              "over all its outputs")
         if self.all_scores and spec.router_bias:
             raise ValueError("the router that scores by the softmax over all its outputs has no bias")
+        if spec.weigh_input and (spec.expert == "gated_clamped" or spec.identity_experts or spec.shared_size):
+            raise ValueError("weights in front of the experts are for experts without clamps, identities and a shared expert")
         self.outputs = spec.experts + spec.identity_experts
         if self.outputs % spec.group_count or spec.group_keep > spec.group_count:
             raise ValueError(f"{self.outputs} router outputs do not form {spec.group_count} equal groups of which "
@@ -165,7 +167,8 @@ class RoutedExperts(Part):
         if not self.all_scores:
             ids, weights = ops.moe_route(x, self.router, self.router_bias, s.top, s.scoring, s.weight_scale)
             self.last_ids = ids
-            return ops.moe_experts(x, ids, weights, self.gate_up, self.down, s.limit, s.expert, status=status)
+            return ops.moe_experts(x, ids, weights, self.gate_up, self.down, s.limit, s.expert, status=status,
+                                   weigh_input=s.weigh_input)
         routed = ops.moe_route_all(x, self.router, self.correction, s.top, s.group_count, s.group_keep, s.weight_scale,
                                    shared_gate=bool(s.shared_size))
         ids, weights = routed[0], routed[1]
@@ -176,7 +179,7 @@ class RoutedExperts(Part):
             shared = ops.linear(act, self.shared_down, status=status)
         return ops.moe_experts(x, ids, weights, self.gate_up, self.down, s.limit, s.expert, status=status,
                                identity=bool(s.identity_experts), shared=shared,
-                               shared_gate=routed[2] if s.shared_size else None)
+                               shared_gate=routed[2] if s.shared_size else None, weigh_input=s.weigh_input)
 
     def weight_bytes(self):
         """What a step reads at most: the router and every expert (a step of few tokens reads only the

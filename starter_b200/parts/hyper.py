@@ -3,7 +3,8 @@
 A token has ``S`` streams ``x_1 .. x_S`` (float32 ``[tokens, S, hidden]``), all equal to its embedding
 at the start.  A sublayer with this part's ``in`` ``[S]``, ``out`` ``[S]`` and ``mix`` ``[S, S]``
 (indexed ``[from, to]``) reads ``u = sum_s in[s] * x_s``, computes ``y = sublayer(norm(u))`` and
-writes every stream from the values before the update: ``x_t = sum_s mix[s, t] * x_s + out[t] * y``.  The
+writes every stream from the values before the update: ``x_t = sum_s mix[s, t] * x_s + out[t] * y``.  With a
+``scale`` ``[hidden]`` (a layer scale) ``y`` is multiplied by it, channel by channel, before it is written.  The
 model's output is the sum of the streams.
 
 The update that closes a sublayer and the read (and norm) that opens the next are one kernel
@@ -30,40 +31,50 @@ class Pending:
 
     def for_kernel(self):
         c = self.connection
-        return self.value, c.mix, c.out, self.bias
+        return self.value, c.mix, c.out, self.bias, c.scale
+
+
+def _fused(norm):
+    """The norm as the stream kernel takes it, or None when it runs as a kernel of its own."""
+    parameters = getattr(norm, "parameters", None)
+    return parameters() if parameters is not None else None
 
 
 class HyperConnection(Part):
     def param_specs(self):
         s = self.spec.streams
-        return {"in": ParamSpec((s,), "stream_weight"), "out": ParamSpec((s,), "stream_weight"),
-                "mix": ParamSpec((s, s), "stream_weight")}
+        out = {"in": ParamSpec((s,), "stream_weight"), "out": ParamSpec((s,), "stream_weight"),
+               "mix": ParamSpec((s, s), "stream_weight")}
+        if self.spec.channel_scale is not None:
+            out["scale"] = ParamSpec((self.spec.channel_scale,), "gain32")
+        return out
 
     def set_params(self, params):
         self.read = params["in"].contiguous()
         self.out = params["out"].contiguous()
         self.mix = params["mix"].contiguous()
+        self.scale = params["scale"].float().contiguous() if self.spec.channel_scale is not None else None
 
     def open(self, streams, pending, norm, dtype):
         """Apply ``pending`` (a ``Pending`` or None) to ``streams`` in place and return this sublayer's
         normed input ``[tokens, hidden]`` in ``dtype``."""
         before = pending.for_kernel() if pending is not None else None
-        fused = getattr(norm, "parameters", None)
+        fused = _fused(norm)
         if fused is not None:
-            return ops.hyper_step(streams, dtype, before, self.read, fused())
+            return ops.hyper_step(streams, dtype, before, self.read, fused)
         return norm(ops.hyper_step(streams, dtype, before, self.read, None))
 
     def weight_bytes(self):
-        return bytes_of(self.read, self.out, self.mix)
+        return bytes_of(self.read, self.out, self.mix, self.scale)
 
 
 def close_rows(streams, pending, rows, norm, dtype):
     """The model's end for the rows asked for: the last pending update, the sum of the streams and the
     final norm, without touching ``streams``."""
     before = pending.for_kernel() if pending is not None else None
-    fused = getattr(norm, "parameters", None)
+    fused = _fused(norm)
     if fused is not None:
-        return ops.hyper_step(streams, dtype, before, None, fused(), rows=rows)
+        return ops.hyper_step(streams, dtype, before, None, fused, rows=rows)
     return norm(ops.hyper_step(streams, dtype, before, None, None, rows=rows))
 
 

@@ -2,6 +2,8 @@
 
 from __future__ import annotations
 
+import torch
+
 from .. import ops
 from .base import ParamSpec, Part, bytes_of
 
@@ -22,6 +24,11 @@ class RMSNorm(Part):
         if getattr(self.spec, "unit_offset", False):
             # stored around zero: the gain is formed once, in float32, and the kernels see a plain gain
             self.weight = (1.0 + self.weight.float()).contiguous()
+
+    def parameters(self):
+        """``(gain, eps)`` for the kernel that reads several residual streams and norms what it read; None when the
+        gain is not held in float32 (the norm then runs as a kernel of its own)."""
+        return (self.weight, self.spec.eps) if self.weight.dtype == torch.float32 else None
 
     def __call__(self, x):
         return ops.rmsnorm(x, self.weight, self.spec.eps)

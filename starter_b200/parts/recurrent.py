@@ -6,11 +6,14 @@ whose last inputs are part of that state:
 * ``StateSpaceMixer``: a selective state-space recurrence with a matrix state per head (``ops.short_conv``,
   ``ops.state_scan`` in its ``state_space`` form, ``ops.group_norm_gate``);
 * ``GatedDeltaMixer``: the gated delta rule on unit queries and keys (the same three kernels, the scan in its
-  ``gated_delta`` form).
+  ``gated_delta`` form);
+* ``ForgetWriteMixer``: a forget gate per key channel that also decides what is written (no convolution; the scan in
+  its ``forget_write`` form, ``ops.group_norm_gate`` without a gate).
 
 A whole prompt, a later portion and a single token are the same code, and a step captured in a CUDA graph too:
 the kernels work from the step's device arrays and the slots.  A slot's floats: the convolution's last ``taps -
-1`` inputs of every convolved channel, then the recurrence's state; zero when a sequence opens.
+1`` inputs of every convolved channel, then the recurrence's state, from ``state_at`` on (another mixer may share
+the slot); zero when a sequence opens.
 """
 
 from __future__ import annotations
@@ -36,6 +39,7 @@ class _Recurrent(Part):
         super().__init__(spec, dtype)
         if position is not None:
             raise ValueError(f"{type(self).__name__} takes no position part")
+        self.state_at = 0
 
     def kv_need(self):
         return None
@@ -88,7 +92,7 @@ class GatedLinearRecurrence(_Recurrent):
         state = self._state(ctx, entry, writes_cache)
         seqs = (ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len, ctx.max_q_len)
         proj = ops.linear(x, self.yx, status=ctx.status)                      # [y | x]
-        u = ops.short_conv(proj, c, c, self.conv, self.conv_bias, self.x_bias, state, 0, *seqs)
+        u = ops.short_conv(proj, c, c, self.conv, self.conv_bias, self.x_bias, state, self.state_at, *seqs)
         parts = u.view(u.shape[0], s.blocks, self.block).transpose(0, 1)
         # the gates' logits stay 32-bit (a library product, as the head-wise products of the latent attention are)
         if u.dtype == torch.float32:
@@ -96,7 +100,7 @@ class GatedLinearRecurrence(_Recurrent):
         else:
             logits = torch.bmm(parts, self.gates, out_dtype=torch.float32)
         out = ops.glru_scan(u, logits, self.ra_bias, self.ri_bias, self.lam, s.decay_scale, proj, 0, self.y_bias,
-                            state, (s.conv - 1) * c, *seqs)
+                            state, self.state_at + (s.conv - 1) * c, *seqs)
         return ops.linear(out, self.o, status=ctx.status)
 
     def weight_bytes(self):
@@ -141,11 +145,11 @@ class StateSpaceMixer(_Recurrent):
         state = self._state(ctx, entry, writes_cache)
         seqs = (ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len)
         proj = ops.linear(x, self.w_in, status=ctx.status)
-        xbc = ops.short_conv(proj, self.inner, self.convolved, self.conv, self.conv_bias, None, state, 0, *seqs,
+        xbc = ops.short_conv(proj, self.inner, self.convolved, self.conv, self.conv_bias, None, state, self.state_at, *seqs,
                              ctx.max_q_len, "silu")
         y = ops.state_scan("state_space", (xbc, self.inner + self.bc), (xbc, self.inner), (xbc, 0),
                            (proj, self.inner + self.convolved), None, self.A_log, self.dt_bias, self.D, state,
-                           (s.conv - 1) * self.convolved, *seqs, s.num_heads, s.groups, s.state, s.head_dim)
+                           self.state_at + (s.conv - 1) * self.convolved, *seqs, s.num_heads, s.groups, s.state, s.head_dim)
         y = ops.group_norm_gate(y, proj, 0, self.gain, s.norm_groups, s.norm_eps, True, x.dtype)
         return ops.linear(y, self.o, status=ctx.status)
 
@@ -191,14 +195,55 @@ class GatedDeltaMixer(_Recurrent):
         state = self._state(ctx, entry, writes_cache)
         seqs = (ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len)
         proj = ops.linear(x, self.stacked, status=ctx.status)
-        qkv = ops.short_conv(proj, 0, self.convolved, self.conv, None, None, state, 0, *seqs, ctx.max_q_len, "silu")
+        qkv = ops.short_conv(proj, 0, self.convolved, self.conv, None, None, state, self.state_at, *seqs, ctx.max_q_len,
+                             "silu")
         gate_at = self.convolved
         beta_at = gate_at + self.inner
         o = ops.state_scan("gated_delta", (qkv, 0), (qkv, self.qk), (qkv, 2 * self.qk), (proj, beta_at + s.num_heads),
-                           (proj, beta_at), self.A_log, self.dt_bias, None, state, (s.conv - 1) * self.convolved, *seqs,
+                           (proj, beta_at), self.A_log, self.dt_bias, None, state,
+                           self.state_at + (s.conv - 1) * self.convolved, *seqs,
                            s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim)
         y = ops.group_norm_gate(o, proj, gate_at, self.gain, s.num_heads, s.norm_eps, False, x.dtype)
         return ops.linear(y, self.o, status=ctx.status)
 
     def weight_bytes(self):
         return bytes_of(self.stacked, self.conv, self.A_log, self.dt_bias, self.gain, self.o)
+
+
+class ForgetWriteMixer(_Recurrent):
+    def __init__(self, spec, dtype, position=None):
+        super().__init__(spec, dtype, position)
+        self.qk = spec.num_heads * spec.head_dim
+        self.inner = spec.num_heads * spec.value_dim
+
+    def state_need(self):
+        s = self.spec
+        return StateNeed((s.num_heads * s.head_dim * s.value_dim,), "float32")
+
+    def param_specs(self):
+        s = self.spec
+        return {
+            "q": ParamSpec((self.qk, s.hidden_size)), "f": ParamSpec((self.qk, s.hidden_size)),
+            "f_bias": ParamSpec((self.qk,), "bias32"), "lower": ParamSpec((self.qk,), "floor"),
+            "v": ParamSpec((self.inner, s.hidden_size)), "norm": ParamSpec((s.value_dim,), "gain32"),
+            "o": ParamSpec((s.hidden_size, self.inner)),
+        }
+
+    def set_params(self, params):
+        self.stacked = _padded_rows([params[n] for n in ("q", "f", "v")], self.spec.hidden_size)      # [q | f | v]
+        self.f_bias, self.lower = params["f_bias"].float().contiguous(), params["lower"].float().contiguous()
+        self.gain = params["norm"].float().contiguous()
+        self.o = params["o"].contiguous()
+
+    def __call__(self, x, ctx, entry, writes_cache=True):
+        s = self.spec
+        state = self._state(ctx, entry, writes_cache)
+        proj = ops.linear(x, self.stacked, status=ctx.status)
+        o = ops.state_scan("forget_write", (proj, 0), (proj, self.qk), (proj, 2 * self.qk), None, None, self.lower,
+                           self.f_bias, None, state, self.state_at, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
+                           s.num_heads, s.num_heads, s.head_dim, s.value_dim)
+        y = ops.group_norm_gate(o, None, 0, self.gain, s.num_heads, s.norm_eps, False, x.dtype)
+        return ops.linear(y, self.o, status=ctx.status)
+
+    def weight_bytes(self):
+        return bytes_of(self.stacked, self.f_bias, self.lower, self.gain, self.o)

@@ -33,7 +33,7 @@ from .feedforward import BiasedFeedForward, ClampedGatedFeedForward, GatedFeedFo
 from .hyper import HyperConnection, HyperMixerOnlyBlock, HyperPreNormBlock
 from .norm import RMSNorm
 from .parallel import ParallelMixer
-from .recurrent import GatedDeltaMixer, GatedLinearRecurrence, StateSpaceMixer
+from .recurrent import ForgetWriteMixer, GatedDeltaMixer, GatedLinearRecurrence, StateSpaceMixer
 from .norm_dyt import DynamicTanh
 from .norm_layer import LayerNorm
 from .rotary import InterleavedRotaryTable, PartialRotaryTable, RotaryTable
@@ -87,4 +87,5 @@ register("arrangement", "prenorm32_mixer_only", PreNorm32MixerOnlyBlock)
 register("mixer", "gated_linear_recurrence", GatedLinearRecurrence)
 register("mixer", "state_space", StateSpaceMixer)
 register("mixer", "gated_delta", GatedDeltaMixer)
+register("mixer", "forget_write", ForgetWriteMixer)
 register("mixer", "parallel", ParallelMixer)

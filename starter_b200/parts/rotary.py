@@ -11,6 +11,7 @@ so that they are the same bits on every machine, and grow on demand.
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 
 import torch
@@ -75,25 +76,49 @@ class InterleavedRotaryTable(RotaryTable):
     def rotation(self) -> Rotation:
         return Rotation(self.cos, self.sin, self.spec.dims, "interleaved")
 
+    def frequencies(self):
+        """``(float64 [dims / 2], multiplier of cos and sin)``."""
+        dims = self.spec.dims
+        i = torch.arange(dims // 2, dtype=torch.float64)
+        return torch.pow(torch.tensor(float(self.spec.base), dtype=torch.float64), -2.0 * i / dims), 1.0
+
     def ensure(self, length: int) -> bool:
         if length <= self.length:
             return False
         size = max(self.MIN_POSITIONS, self.length)
         while size < length:
             size *= 2
-        dims = self.spec.dims
-        i = torch.arange(dims // 2, dtype=torch.float64)
-        freq = torch.pow(torch.tensor(float(self.spec.base), dtype=torch.float64), -2.0 * i / dims)
+        freq, mult = self.frequencies()
         angles = torch.outer(torch.arange(size, dtype=torch.float64), freq)
-        self.cos = angles.cos().float().contiguous().to(self.device)
-        self.sin = angles.sin().float().contiguous().to(self.device)
+        self.cos = (angles.cos() * mult).float().contiguous().to(self.device)
+        self.sin = (angles.sin() * mult).float().contiguous().to(self.device)
         self.length = size
         return True
 
 
 class PartialRotaryTable(InterleavedRotaryTable):
     """Tables for a rotation of entry ``i`` with entry ``i + dims / 2`` over the first ``dims`` entries of a
-    vector: the same angles ``position * base ** (-2i / dims)`` as the interleaved tables, paired half-split."""
+    vector: the same angles ``position * base ** (-2i / dims)`` as the interleaved tables, paired half-split.  The
+    spec's ``scaling`` changes the frequencies (and, for YaRN, multiplies cos and sin)."""
+
+    def frequencies(self):
+        freq, mult = super().frequencies()
+        scaling = self.spec.scaling
+        if scaling is None:
+            return freq, mult
+        if not hasattr(scaling, "original"):
+            return freq / scaling.factor, mult
+        dims, base = self.spec.dims, float(self.spec.base)
+
+        def index_of(turns: float) -> float:
+            # the (fractional) frequency that makes that many turns over the original length
+            return dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo = max(math.floor(index_of(scaling.fast)), 0)
+        hi = min(math.ceil(index_of(scaling.slow)), dims - 1)
+        i = torch.arange(dims // 2, dtype=torch.float64)
+        stretched = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return freq / scaling.factor * stretched + freq * (1.0 - stretched), 0.1 * math.log(scaling.factor) + 1.0
 
     def rotation(self) -> Rotation:
         return Rotation(self.cos, self.sin, self.spec.dims, "half_split")
