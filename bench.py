@@ -903,6 +903,112 @@ def bavedra_compare(args) -> int:
                               beside=("kesedra", "Kesedra", kesedra_config, kesedra_kernels_alone))
 
 
+def setotar_config(size: dict, layers: int) -> dict:
+    """Setotar at ``size``: of every four layers an attention over all keys (its queries and keys normed over their
+    rows, 64 of 128 entries rotated, stretched by parts), two window attentions of 1,024 keys that keep the first four,
+    with biases, three taps, unit values and capped scores, each beside a forget-write recurrence with states of 128 x
+    128, and an attention that reads the first one's keys and values; four streams; 16 experts of a quarter of the
+    dense width, four a token, in every layer."""
+    w, out = size["width"], []
+    moe = dict(kind="moe", expert=dict(ff=size["ff"] // 4 // 64 * 64), router=dict(experts=16, top=4))
+    heads = dict(heads=size["heads"], kv_heads=size["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5)
+    full = dict(heads, rot=dict(base=1e6, dims=64, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)))
+    side = dict(left=dict(heads, conv=3, mask=dict(size=1024, keep_first=4), softcap=50.0,
+                          rot=dict(base=1e4, dims=64, scaling=dict(factor=2.0))),
+                right=dict(heads=w // 128, dim=128, vdim=128), left_scale=0.6, right_scale=0.5)
+    for i in range(layers):
+        if i % 4 in (1, 2):
+            out.append(dict(type="parallel", mixer=side, mlp=moe))
+        else:
+            out.append(dict(type="attention", mixer=full if i % 4 == 0 else dict(full, kv_from=i - 3), mlp=moe))
+    return dict(architecture="Setotar", vocab=size["vocab"], width=w, streams=4, norm=dict(eps=1e-6), layers=out)
+
+
+def setotar_kernels_alone(ops, out, name, rows, x, blocks, spec, cache, ctx, size, batch, context, prompt_len, rnd,
+                          in_graph, bw, tc):
+    """Setotar's own kernels alone at ``rows`` rows, once per layer inside a CUDA graph."""
+    import torch
+
+    w, dev, bf, n_streams = size["width"], x.device, x.dtype, spec.streams
+    streams = torch.randn(rows, n_streams, w, device=dev) * 0.1
+    us = in_graph([lambda b=b: ops.hyper_step(streams, bf, (x, b.connection1.mix * 0.1, b.connection1.out, None, b.connection1.scale),
+                                              b.connection1.read, b.norm1.parameters()) for b in blocks])
+    out[f"{name}: stream write, read + norm ({n_streams} streams)"] = bw(us, rows * w * (2 + 8 * n_streams + 2))
+    seqs = (ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len)
+    n_seqs = ctx.n_seqs
+    pairs = [(b, e) for b, e in zip(blocks, spec.schedule)]
+
+    def attention(title, chosen, a_of):
+        a = a_of(chosen[0][0])
+        sp = a.spec
+        heads, kvh, dim, vdim = sp.num_heads, sp.num_kv_heads, sp.head_dim, sp.value_dim
+        proj = rnd(rows, a.qkvg.shape[0])
+        if a.taps is not None:
+            us = in_graph([lambda b=b, e=e: ops.short_conv(proj, 0, a.convolved, a_of(b).taps, None, a_of(b).biases, cache.entry_state(e.cache),
+                                                            a_of(b).state_at, *seqs, ctx.max_q_len) for b, e in chosen])
+            state = n_seqs * (sp.conv - 1) * a.convolved * 8
+            out[f"{name}: bias + short convolution ({a.convolved} channels)"] = bw(us, rows * a.convolved * 4 + state)
+
+        def prepare(b, e):
+            k, v = cache.entry_pages(e.cache)
+            ops.sink_prepare_half(proj, heads, kvh, dim, vdim, ctx.tok_pos, ctx.tok_slot, cache.block_table, k, v,
+                                  a.position.rotation(), a_of(b).row_norm, sp.unit_values, sp.norm_eps)
+
+        def attend(b, e):
+            k, v = cache.entry_pages(e.cache)
+            return ops.sink_attention_step(proj, k, v, cache.block_table, ctx, heads, kvh, dim, vdim, sp.scale, None, None, None, None,
+                                           sp.window, sp.keep_first, sp.softcap)
+
+        us = in_graph([lambda b=b, e=e: prepare(b, e) for b, e in chosen])
+        turned = 2 * heads * dim if sp.row_norm else heads * sp.position.dims * 2
+        out[f"{name}: {title}: norms, rotation, cache write"] = bw(us, rows * 2 * (turned + 2 * kvh * (dim + vdim)))
+        us = in_graph([lambda b=b, e=e: attend(b, e) for b, e in chosen])
+        span = lambda p: p + 1 if sp.window is None else min(p + 1, sp.window + sp.keep_first)  # noqa: E731
+        if rows == prompt_len:
+            out[f"{name}: {title}: attention"] = tc(us, heads * 2 * (dim + vdim) * sum(span(p) for p in range(prompt_len)))
+        else:
+            out[f"{name}: {title}: attention"] = bw(us, batch * span(context) * kvh * (dim + vdim) * 2)
+
+    attention("all keys", [(b, e) for b, e in pairs if b.mixer.spec.kind == "sink_attention" and e.writes_cache], lambda b: b.mixer)
+    par = [(b, e) for b, e in pairs if b.mixer.spec.kind == "parallel"]
+    attention("window, kept keys, cap", par, lambda b: b.mixer.sides["left"])
+    m = par[0][0].mixer.sides["right"]
+    sp = m.spec
+    proj = rnd(rows, m.stacked.shape[0])
+    us = in_graph([lambda b=b, e=e: ops.state_scan("forget_write", (proj, 0), (proj, m.qk), (proj, 2 * m.qk), None, None,
+                                                    b.mixer.sides["right"].lower, b.mixer.sides["right"].f_bias, None,
+                                                    cache.entry_state(e.cache), b.mixer.sides["right"].state_at, *seqs, sp.num_heads,
+                                                    sp.num_heads, sp.head_dim, sp.value_dim) for b, e in par])
+    d = bw(us, rows * (2 * m.qk * 2 + m.inner * 6) + n_seqs * sp.num_heads * sp.head_dim * sp.value_dim * 4 * 2)
+    d["gflops"] = rows * sp.num_heads * sp.head_dim * sp.value_dim * 5 / us / 1e3
+    out[f"{name}: forget-write recurrence (gate, state walk)"] = d
+    o32 = torch.randn(rows, m.inner, device=dev)
+    us = in_graph([lambda b=b: ops.group_norm_gate(o32, None, 0, b.mixer.sides["right"].gain, sp.num_heads, 1e-6, False, bf)
+                   for b, _ in par])
+    out[f"{name}: head norm"] = bw(us, rows * m.inner * (4 + 2))
+    us = in_graph([lambda b=b: ops.scaled_sum(x, x, 0.6, 0.5) for b, _ in par])
+    out[f"{name}: scaled sum of two mixers"] = bw(us, rows * w * 2 * 3)
+    ff = blocks[0].feed_forward
+    fs = ff.spec
+    ids, weights = ops.moe_route(x, ff.router, None, fs.top, fs.scoring)
+    us = in_graph([lambda b=b: ops.moe_route(x, b.feed_forward.router, None, fs.top, fs.scoring) for b in blocks])
+    out[f"{name}: router"] = bw(us, rows * w * 2 + ff.router.shape[0] * w * 4)
+    us = in_graph([lambda b=b: ops.moe_experts(x, ids, weights, b.feed_forward.gate_up, b.feed_forward.down, 0.0, "gated_silu",
+                                               weigh_input=True) for b in blocks])
+    if rows == prompt_len:
+        out[f"{name}: experts (gate, up, down, sum)"] = tc(us, rows * fs.top * 3 * fs.intermediate_size * w * 2)
+    else:
+        used = int(torch.unique(ids).numel())
+        out[f"{name}: experts (gate, up, down, sum)"] = bw(us, used * 3 * fs.intermediate_size * w * 2)
+
+
+def setotar_compare(args) -> int:
+    """Beside Bavedra: the closest design this library has (a window attention beside a recurrence with a matrix state
+    per head, rotated keys, routed experts, a 32-bit residual)."""
+    return compare_with_qwen3(args, "setotar", "Setotar", setotar_config, setotar_kernels_alone, ["2048"],
+                              beside=("bavedra", "Bavedra", bavedra_config, bavedra_kernels_alone))
+
+
 def kesedra_compare(args) -> int:
     # the 2048 size alone by default: at 2560 with 8 layers a prompt step of this design failed to return while
     # its kernels still released their successors early; the larger sizes have not been timed since and run
@@ -915,7 +1021,7 @@ def korurax_compare(args) -> int:
 
 
 def compare_with_qwen3(args, design_key, design_title, config_of, own_kernels, default_sizes, beside=None) -> int:
-    """``--design kesedra`` / ``korurax`` / ``bavedra``: prefill and decode throughput of that design beside Qwen3
+    """``--design kesedra`` / ``korurax`` / ``bavedra`` / ``setotar``: prefill and decode throughput of that design beside Qwen3
     (or, with ``beside = (key, title, config_of, kernels_alone)``, beside that design: the closest model this library
     has) at equal width, dense feed-forward, vocabulary and head count, and the design's own kernels alone beside the
     other's like kernels, each against its roofline.  Every number is timed on the device with CUDA events; the
@@ -1078,8 +1184,8 @@ def main() -> int:
                              "generation range); the cache is sized for it")
     parser.add_argument("--per-stage", action="store_true",
                         help="also print where a decode step's time goes, kernel by kernel (stderr)")
-    parser.add_argument("--design", choices=["goguvik", "kesedra", "korurax", "bavedra"], default=None,
-                        help="instead of the default run: that design beside Qwen3 (Bavedra: beside Kesedra) at equal "
+    parser.add_argument("--design", choices=["goguvik", "kesedra", "korurax", "bavedra", "setotar"], default=None,
+                        help="instead of the default run: that design beside Qwen3 (Bavedra: Kesedra; Setotar: Bavedra) at equal "
                              "sizes (prefill, decode, and each design's own kernels against their rooflines)")
     parser.add_argument("--design-sizes", default=None, help="comma-separated subset of " + ",".join(DESIGN_SIZES))
     args = parser.parse_args()
@@ -1093,6 +1199,8 @@ def main() -> int:
         return workload(args)
     if args.design == "korurax":
         return korurax_compare(args)
+    if args.design == "setotar":
+        return setotar_compare(args)
     if args.design == "bavedra":
         return bavedra_compare(args)
     if args.design == "kesedra":

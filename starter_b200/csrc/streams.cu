@@ -151,7 +151,8 @@ __global__ void hyper_step_kernel(float* __restrict__ streams, const T* __restri
 // The same with an RMS norm of u: a block takes a whole row, whose u waits in shared memory (hidden floats) for
 // the sum of squares.
 template <typename T, int S, int V>
-__global__ void hyper_rms_kernel(float* __restrict__ streams, const T* __restrict__ y, const float* __restrict__ y_bias,
+__global__ void __launch_bounds__(S <= 4 ? 512 : 256)
+hyper_rms_kernel(float* __restrict__ streams, const T* __restrict__ y, const float* __restrict__ y_bias,
                                  const float* __restrict__ y_scale, const float* __restrict__ mix_prev,
                                  const float* __restrict__ out_prev, const float* __restrict__ in_next,
                                  const float* __restrict__ gain, float eps, T* __restrict__ normed,
@@ -275,7 +276,7 @@ static int launch_step_v(int S, float* streams, const void* y, const float* y_bi
                          int n_rows, int hidden, cudaStream_t s) {
   if (norm_kind == 2) {
     const int pieces = (hidden + V - 1) / V;
-    const int threads = pieces >= 1024 ? 512 : pieces > 128 ? 256 : 128;
+    const int threads = pieces >= 1024 && S <= 4 ? 512 : pieces > 128 ? 256 : 128;
     const size_t smem = (size_t)hidden * sizeof(float);
     if (smem > 51200 * sizeof(float)) return -2;
 #define GO(N) case N: {                                                                                                  \

@@ -95,14 +95,17 @@ def rotate(x, positions, rot):
 
 
 def visible(i, j, window=None, keep_first=0):
-    return j <= i and (window is None or i - j < window or j < keep_first)
+    """Whether query ``i`` sees key ``j`` (tensors of positions)."""
+    if window is None:
+        return j <= i
+    return (j <= i) & ((i - j < window) | (j < keep_first))
 
 
 def attend(q, k, v, scale, cap=None, window=None, keep_first=0):
     """``q`` ``[T, H, D]``, ``k`` ``[T, G, D]``, ``v`` ``[T, G, V]`` -> ``[T, H, V]``."""
     T, H, _ = q.shape
     G = k.shape[1]
-    seen = torch.tensor([[visible(i, j, window, keep_first) for j in range(T)] for i in range(T)])
+    seen = visible(torch.arange(T)[:, None], torch.arange(T)[None, :], window, keep_first)
     out = torch.zeros((T, H, v.shape[-1]), dtype=q.dtype)
     for h in range(H):
         g = h // (H // G)

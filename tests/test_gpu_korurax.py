@@ -289,13 +289,13 @@ def test_attention_alone_with_one_key_that_stands_out(heads, kv_heads, dim, vdim
     for blocks in ((ints([0, 0]), ints([0, 256])), None):
         out = ops.sink_attention_tcgen05(q2, ks, vs, table, ints([1]), ints([0]), ints([n]), ints([n]), ints([0, 0, 0, 0, 0]),
                                          ints([128, 0, 256, 192, 64]), heads, kv_heads, dim, scale, pen, sk, gt, chunk, window,
-                                         status, blocks)
+                                         status, blocks, vdim)
         close(out, want, dtype, "tcgen05, whole")
     late = torch.arange(130, 300, device="cuda")
     out = ops.sink_attention_tcgen05(q2[late].contiguous(), ks, vs, table, ints([1]), ints([0]), ints([170]), ints([n]),
                                      ints([0, 0, 0]), ints([0, 64, 128]), heads, kv_heads, dim, scale, pen, sk,
                                      gt[late].contiguous() if gt is not None else None, chunk, window, status,
-                                     (ints([0]), ints([0])))
+                                     (ints([0]), ints([0])), vdim)
     close(out, want[130:], dtype, "tcgen05, a later portion")
     assert int(status.item()) == 0
 
