@@ -32,8 +32,9 @@
 // sequence's first keys visible, whose pages then come in front of the window's in the walk.  The queries may
 // lie at the front of wider rows (a stacked projection): the tensor map of Q covers those rows.
 // Keys and values have sizes of their own there, up to 128 each, in shared-memory tiles of one or two 64-entry
-// chunks: S runs over the keys' real entries; V's entries behind the real ones arrive as the zeros TMA fills in,
-// and the output columns they give are not stored.
+// chunks.  Entries of a key or a value behind the real ones arrive as the zeros TMA fills in: they take what lies
+// behind a query's own entries (its neighbour's) out of S, and the output columns they give are not stored.
+// (Loops over the real sizes would make the one lane that issues the products form every descriptor anew.)
 //
 // Every wait on an mbarrier gives up after WAIT_LIMIT_NS, raises bit 16 of *status and lets the
 // block drain its copies, free its tensor memory and return.
@@ -230,7 +231,8 @@ struct TcExtras {
   int dim, vdim;
 };
 
-template <int DC, int VC, bool EXT>
+// EXT 0: plain; 1: the extras without the cap; 2: all of them.
+template <int DC, int VC, int EXT>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -241,6 +243,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             int heads, int kv_heads, float scale_log2, int window, int* status, int list_of_blocks,
                             TcExtras ex) {
   // DC, VC: 64-element (128-byte) chunks of a key and of a value
+  constexpr bool CAP = EXT == 2;
   const int dim = EXT ? ex.dim : DC * 64, vdim = EXT ? ex.vdim : VC * 64;
   constexpr int SUB = 128 * 128;                    // bytes of a [128 rows x 128 bytes] sub-tile
   constexpr int Q_BYTES = DC * SUB;                 // one tile of 128 queries
@@ -357,14 +360,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (n_mine > 0) {
       // the whole warp waits and computes descriptors; one elected lane issues (see the producer)
       const bool elected = elect_one();
-      const uint32_t idesc_s = instr_desc(TC_BK, 0), idesc_o = instr_desc((vdim + 15) & ~15, 1);
+      const uint32_t idesc_s = instr_desc(TC_BK, 0), idesc_o = instr_desc(VC * 64, 1);
       const uint32_t q_addr = smem_u32(q_sm + t * Q_BYTES), p_addr = smem_u32(p_sm + t * P_BYTES);
       // S = Q K^T: k runs over the head in steps of 16 (32 bytes inside a 128-byte chunk)
       auto issue_s = [&](int buf) {
         if (elected) {
 #pragma unroll
           for (int k = 0; k < DC * 4; ++k) {
-            if (EXT && k * 16 >= dim) break;
             const uint32_t off = (k >> 2) * SUB + (k & 3) * 32;
             umma_bf16(tmem_base + t * TC_BK, smem_desc(q_addr + off, 16),
                       smem_desc(smem_u32(ring + buf * KV_BYTES) + off, 16), idesc_s, k > 0 ? 1u : 0u);
@@ -455,6 +457,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         l_run = 1.f;
       }
     }
+    const int row_first = max(row_lo, window > 0 ? pos - window + 1 : 0);
+    const uint32_t gap = EXT ? (uint32_t)max(row_first - ex.keep, 0) : 0u;
+    float series[6];
+    if (CAP) cap_series(ex.cap_in, ex.cap_out, series);
     pdl_wait();
     bool ok = true;
     for (int i = 0; i < n_mine && ok; ++i) {
@@ -473,10 +479,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
       auto load_half = [&](int h) {
         tmem_load64(tmem_s + h * 64, sv);
         const int j0 = h ? jp[1] : jp[0];
-        if (EXT && ex.cap_out > 0.f) {
-#pragma unroll
-          for (int e = 0; e < 64; ++e) sv[e] = ex.cap_out * tanh_fast(sv[e] * ex.cap_in);
-        }
+        if (CAP) cap64(sv, ex.cap_in, ex.cap_out, series);
         if (EXT && ex.r1) {
           const float far = (float)(pos - j0);                // the distance to this half's first key
 #pragma unroll
@@ -487,7 +490,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
           for (int e = 0; e < 64; ++e) {
             const int j = j0 + e;
-            if (j > pos || (((window > 0 && j <= pos - window) || (EXT && j < row_lo)) && !(EXT && j < ex.keep))) sv[e] = -INFINITY;
+            if constexpr (EXT != 0) {
+              // hidden: what comes later, and the gap between the kept keys and the row's first key (without a
+              // branch: the nested conditions compiled to branches doubled the time of a windowed prompt)
+              if ((j > pos) | ((uint32_t)(j - ex.keep) < gap)) sv[e] = -INFINITY;
+            } else if (j > pos || (window > 0 && j <= pos - window)) {
+              sv[e] = -INFINITY;
+            }
           }
         }
       };
@@ -622,7 +631,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 
 // ------------------------------------------------------------------------------------------ host
 
-template <int DC, int VC, bool EXT>
+template <int DC, int VC, int EXT>
 static int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, void* out,
                   const int* block_table, int table_stride, const int* seq_slot, const int* seq_q_start,
                   const int* seq_q_len, const int* seq_kv_len, const int* tile_seq, const int* tile_first,
@@ -684,7 +693,7 @@ int sb_attention_prefill_tc(const void* q, void* out, const void* k_store, const
     cudaMemcpyToSymbolAsync(tc_wait_limit_ns, &next_limit_ns, sizeof(next_limit_ns), 0, cudaMemcpyHostToDevice, s);
     cudaStreamSynchronize(s);
   }
-  rc = head_dim == 64 ? launch<1, 1, false>(ARGS) : launch<2, 2, false>(ARGS);
+  rc = head_dim == 64 ? launch<1, 1, 0>(ARGS) : launch<2, 2, 0>(ARGS);
   if (test_run) {
     cudaStreamSynchronize(s);
     next_withhold_step = -1;
@@ -724,8 +733,10 @@ int sb_sink_attention_tcgen05(const void* q, int q_width, void* out, const void*
                     cap > 0.f ? scale / cap : 0.f, cap > 0.f ? cap / scale : 0.f, dim, vdim};
 #define ARGS mq, mk, mv, out, block_table, table_stride, seq_slot, seq_q_start, seq_q_len, seq_kv_len, tile_seq, \
              tile_first, n_tiles, heads, kv_heads, scale, window, status, list_of_blocks, s, ex
-  if (dim <= 64) return vdim <= 64 ? launch<1, 1, true>(ARGS) : launch<1, 2, true>(ARGS);
-  return vdim <= 64 ? launch<2, 1, true>(ARGS) : launch<2, 2, true>(ARGS);
+  const int kind = (dim > 64) * 2 + (vdim > 64);
+  if (ex.cap_out == 0.f)
+    return kind == 0 ? launch<1, 1, 1>(ARGS) : kind == 1 ? launch<1, 2, 1>(ARGS) : kind == 2 ? launch<2, 1, 1>(ARGS) : launch<2, 2, 1>(ARGS);
+  return kind == 0 ? launch<1, 1, 2>(ARGS) : kind == 1 ? launch<1, 2, 2>(ARGS) : kind == 2 ? launch<2, 1, 2>(ARGS) : launch<2, 2, 2>(ARGS);
 #undef ARGS
 }
 

@@ -173,7 +173,7 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
                                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
                                          const float* __restrict__ q_gain, const float* __restrict__ k_gain, float eps,
                                          int unit_v, int heads, int kv_heads, int dim, int vdim, int write) {
-  __shared__ float scratch[33];
+  __shared__ float2 shares[32];
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(proj);
   SB_BEHIND_WAIT(tok_pos);
@@ -186,14 +186,15 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
   const int pos = tok_pos[row], half = rot / 2, pieces = dim / V;
   const float* cr = cos_t + (size_t)pos * half;
   const float* sr = sin_t + (size_t)pos * half;
-  auto inverse_rms = [&](const T* x, int n) {
+  const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  auto squares = [&](const T* x, int n) {                // this thread's share of a row's sum of squares
     float sq = 0.f, f[V];
     for (int c = tid * V; c < n; c += blockDim.x * V) {
       sink_load<T, V>(x + c, f);
 #pragma unroll
       for (int i = 0; i < V; ++i) sq += f[i] * f[i];
     }
-    return 1.f / sqrtf(block_sum(sq, scratch) / (float)n + eps);
+    return sq;
   };
   // piece c of a head: normed, turned with its partner (which this thread handles too) and stored
   auto turn = [&](const T* from, T* to, const float* gain, float inv, int c) {
@@ -223,8 +224,19 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
     sink_store<T, V>(to + at, g);
     sink_store<T, V>(to + half + at, y);
   };
-  const float q_inv = q_gain ? inverse_rms(q, heads * dim) : 1.f;
-  const float k_inv = k_gain && write ? inverse_rms(k, kv_heads * dim) : 1.f;
+  float q_inv = 1.f, k_inv = 1.f;
+  if (q_gain) {
+    const float mine_q = warp_sum(squares(q, heads * dim)), mine_k = write ? warp_sum(squares(k, kv_heads * dim)) : 0.f;
+    if (lane == 0) shares[warp] = make_float2(mine_q, mine_k);
+    __syncthreads();
+    float sq = 0.f, sk = 0.f;
+    for (int i = 0; i < warps; ++i) {
+      sq += shares[i].x;
+      sk += shares[i].y;
+    }
+    q_inv = 1.f / sqrtf(sq / (float)(heads * dim) + eps);
+    k_inv = 1.f / sqrtf(sk / (float)(kv_heads * dim) + eps);
+  }
   for (int e = tid; e < heads * pieces; e += blockDim.x) {
     const int h = e / pieces, c = e - h * pieces;
     if (!q_gain && c * V >= half) continue;             // queries in place: nothing to do for entries that stay
@@ -238,7 +250,6 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
     turn(k + (size_t)h * dim, k_store + page_row(page, h, off, kv_heads, dim), k_gain ? k_gain + (size_t)h * dim : nullptr,
          k_inv, c);
   }
-  const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
   for (int h = warp; h < kv_heads; h += warps) {
     const T* from = v + (size_t)h * vdim;
     T* to = v_store + page_row(page, h, off, kv_heads, vdim);
@@ -429,7 +440,7 @@ int sb_sink_prepare_half(int dtype, void* proj, int proj_width, const int* tok_p
                          const float* sin_t, int rot, const float* q_gain, const float* k_gain, float eps, int unit_v,
                          int n_tokens, int heads, int kv_heads, int dim, int vdim, int write, cudaStream_t s) {
   if (n_tokens == 0) return 0;
-  if (rot < 0 || rot % 2 || rot > dim || (k_gain && !q_gain)) return -2;
+  if (rot < 0 || rot % 2 || rot > dim || (write && (k_gain != nullptr) != (q_gain != nullptr))) return -2;
   if (proj_width < heads * dim + (write ? kv_heads * (dim + vdim) : 0)) return -2;
 #define HALF_ARGS proj, proj_width, tok_pos, tok_slot, block_table, table_stride, k_store, v_store, cos_t, sin_t, rot, q_gain, \
                   k_gain, eps, unit_v, n_tokens, heads, kv_heads, dim, vdim, write, s

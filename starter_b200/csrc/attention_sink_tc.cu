@@ -184,7 +184,9 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
       sk_ldm4(sk_smem(q_tile + sk_offset<D>(r, 2 * kk + (lane >> 4))), qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
   }
   // ---- this thread's two rows: where they stand, which head they are, what they may see
-  int row_pos[2], row_lo[2], row_head[2], row_pen[2];
+  // (hidden are the keys behind the row's position and the gap between the kept keys and the row's first key)
+  int row_pos[2], row_head[2], row_pen[2];
+  uint32_t row_gap[2];
   float m_run[2], l_run[2];
   bool row_ok[2];
 #pragma unroll
@@ -197,7 +199,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     int first = 0;
     if (chunk > 0) first = row_pos[h] / chunk * chunk;
     if (window > 0 && row_pos[h] - window + 1 > first) first = row_pos[h] - window + 1;
-    row_lo[h] = first;
+    row_gap[h] = (uint32_t)max(first - keep, 0);
     row_pen[h] = (rr % group) * 128 + rr / group + 63;
     const bool with_sink = sink != nullptr && split == 0 && (!share_keys || warp == 0);
     m_run[h] = with_sink ? sink[row_head[h]] * 1.4426950408889634f : -INFINITY;
@@ -232,7 +234,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
           const int jj = warp * 16 + nb * 8 + (lane & 3) * 2 + (e & 1);
           float v = cap_out > 0.f ? cap_out * tanh_fast(s2[nb][e] * cap_in) : s2[nb][e] * scale_log2;
           if (r1) v -= pen_tab[row_pen[h] - jj];
-          if (j0 + jj > row_pos[h] || (j0 + jj < row_lo[h] && j0 + jj >= keep)) v = -INFINITY;
+          if ((j0 + jj > row_pos[h]) | ((uint32_t)(j0 + jj - keep) < row_gap[h])) v = -INFINITY;
           s2[nb][e] = v;
           mx[h] = fmaxf(mx[h], v);
         }
@@ -298,7 +300,7 @@ sink_attention_tc_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         const int jj = nb * 8 + (lane & 3) * 2 + (e & 1);
         float v = cap_out > 0.f ? cap_out * tanh_fast(s[nb][e] * cap_in) : s[nb][e] * scale_log2;
         if (r1) v -= pen_tab[row_pen[h] - jj];
-        if (edge && (j0 + jj > row_pos[h] || (j0 + jj < row_lo[h] && j0 + jj >= keep))) v = -INFINITY;
+        if (edge && ((j0 + jj > row_pos[h]) | ((uint32_t)(j0 + jj - keep) < row_gap[h]))) v = -INFINITY;
         s[nb][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }

@@ -13,7 +13,8 @@
 // new sequence.  Everything but the loads of q, k, v, a_raw, b_raw (working type T) is float; o is stored float.
 //
 // A block owns 32 columns of one head's S for one sequence: 256 threads = 32 columns x 8 lanes; lane p of a
-// column keeps rows p, p + 8, ... (KPT of them) in registers, and the eight lanes of a column sum S^T k and
+// column keeps KPT rows in registers (rows 4p .. 4p + 3 of every 32, so that a token's keys and queries are read from
+// shared memory four at a time; with fewer than four rows a lane, p, p + 8), and the eight lanes of a column sum S^T k and
 // S^T q by shuffles.  (States of more than 64 rows: 16 columns x 16 lanes.)  Both are taken from the state as the
 // token finds it: with u the token's write, (g S + k u^T)^T q = g S^T q + u (k . q), so one round of shuffles a token
 // serves both and the decay is folded into the write.  In mode 2 the write needs no read-out: S moves by d (v - S)
@@ -48,6 +49,23 @@ template <int P> __device__ __forceinline__ float sum_lanes(float v) {
 template <int NP, int COLS> struct ScanBuffer {
   float q[SCAN_CT][NP], k[SCAN_CT][NP], v[SCAN_CT][COLS], dec[SCAN_CT], fac[SCAN_CT], kq[SCAN_CT];   // dec: 1 - decay
 };
+
+// The row of S that register r of lane p holds, and a lane's KPT entries of a token's vector of NP.
+template <int KPT, int P> __device__ __forceinline__ int row_of(int p, int r) {
+  return KPT >= 4 ? (r / 4) * (4 * P) + 4 * p + r % 4 : p + P * r;
+}
+template <int KPT, int P> __device__ __forceinline__ void lane_rows(const float* x, int p, float* out) {
+  if (KPT >= 4) {
+#pragma unroll
+    for (int c = 0; c < KPT / 4; ++c) {
+      const float4 v = *reinterpret_cast<const float4*>(x + c * (4 * P) + 4 * p);
+      out[4 * c] = v.x; out[4 * c + 1] = v.y; out[4 * c + 2] = v.z; out[4 * c + 3] = v.w;
+    }
+  } else {
+#pragma unroll
+    for (int r = 0; r < KPT; ++r) out[r] = x[p + P * r];
+  }
+}
 
 template <typename T, int MODE, int KPT, int P>
 __global__ void __launch_bounds__(256)
@@ -86,7 +104,7 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
   float S[KPT];
 #pragma unroll
   for (int r = 0; r < KPT; ++r) {
-    const int i = p + P * r;
+    const int i = row_of<KPT, P>(p, r);
     S[r] = (col && i < N) ? sp[(size_t)i * V + j] : 0.f;
   }
   // mode 2: A_log holds the lower bounds and dt_bias the biases, [H][N] each; a thread always files the same row of S
@@ -127,7 +145,7 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
 #pragma unroll
     for (int n = 0; n < QK_PER; ++n) {
       const int e = tid + 256 * n;
-      if (e < SCAN_CT * NP) {
+      if (e < SCAN_CT * NP && (MODE != 2 || e < ct * NP)) {      // (mode 2: no gates for tokens that are not there)
         const float qe = to_f<T>(rq[n]), ke = to_f<T>(rk[n]);
         (&b.q[0][0])[e] = MODE == 2 ? qe / (1.f + expf(-qe)) : qe;
         (&b.k[0][0])[e] = MODE == 2 ? rate / (1.f + expf(ke + bias)) : ke;
@@ -181,12 +199,14 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
         part[i] = 0.f;
         if (tb + i < ct) {
           const float x = b.v[tb + i][jj];
-          float ra2 = 0.f, rb2 = 0.f;
+          float kk[KPT], qv[KPT], ra2 = 0.f, rb2 = 0.f;
+          lane_rows<KPT, P>(b.k[tb + i], p, kk);
+          lane_rows<KPT, P>(b.q[tb + i], p, qv);
 #pragma unroll
           for (int r = 0; r < KPT; ++r) {
-            S[r] = fmaf(b.k[tb + i][p + P * r], x - S[r], S[r]);
-            const float s = S[r] * b.q[tb + i][p + P * r];
-            if (r & 1) rb2 += s; else ra2 += s;
+            S[r] = fmaf(kk[r], x - S[r], S[r]);
+            if (r & 1) rb2 += S[r] * qv[r];
+            else ra2 += S[r] * qv[r];
           }
           part[i] = ra2 + rb2;
         }
@@ -208,11 +228,12 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
       // (the decay g arrives as d = 1 - g and is applied as S - d * S: a g close to one, rounded to a float,
       // would lose up to 2^-24 / (1 - g) of the decay's rate)
       const float dd = b.dec[tt], x = b.v[tt][jj];
-      float kk[KPT], r1a = 0.f, r1b = 0.f, r2a = 0.f, r2b = 0.f;
+      float kk[KPT], qv[KPT], r1a = 0.f, r1b = 0.f, r2a = 0.f, r2b = 0.f;
+      lane_rows<KPT, P>(b.k[tt], p, kk);
+      lane_rows<KPT, P>(b.q[tt], p, qv);
 #pragma unroll
       for (int r = 0; r < KPT; ++r) {
-        kk[r] = b.k[tt][p + P * r];
-        const float qq = b.q[tt][p + P * r];
+        const float qq = qv[r];
         if (r & 1) {
           if (MODE == 1) r1b += S[r] * kk[r];
           r2b += S[r] * qq;
@@ -244,7 +265,7 @@ state_scan_kernel(const T* __restrict__ q, int ldq, const T* __restrict__ k, int
   }
 #pragma unroll
   for (int r = 0; r < KPT; ++r) {
-    const int i = p + P * r;
+    const int i = row_of<KPT, P>(p, r);
     if (col && i < N) sp[(size_t)i * V + j] = S[r];
   }
 }
