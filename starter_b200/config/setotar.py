@@ -5,8 +5,8 @@ scaled per channel in front of the write; pre-norm sublayers (RMS norms with pla
 mixers (``attention``: grouped-query attention over all keys, queries and keys normed over their whole projections and
 turned by rotary positions; a layer with ``kv_from: j`` attends over layer ``j``'s keys and values; ``parallel``:
 window attention that keeps the first tokens, with biases, short convolutions, unit-RMS values and capped scores,
-side by side with a linear recurrence whose forget gate also decides what is written, joined as a scaled sum) and a
-mixture of gated experts whose weights (plain sigmoids of the router) multiply their inputs, or no feed-forward.  A
+side by side with a linear recurrence in which one gate a channel sets what is kept and what is written, joined as a
+scaled sum) and a mixture of gated experts, each run on the row times its plain sigmoid, or no feed-forward.  A
 final norm over the sum of the streams and an output head.
 
 ``config.json`` gives ``architecture``, ``vocab``, ``width``, ``streams``, ``norm.eps`` and a list ``layers``; a layer

@@ -176,12 +176,12 @@ class SinkAttentionSpec:
     key/value head's value is its key as projected, before any rotation (``value_dim`` = ``head_dim``).
 
     Further, for layers without head gates: ``keep_first`` (with ``window``): the sequence's first that many keys stay
-    visible however far behind they are, at their true positions.  ``softcap``: a scaled score ``s`` becomes ``softcap *
+    visible however far behind they are.  ``softcap``: a scaled score ``s`` becomes ``softcap *
     tanh(s / softcap)`` before the softmax.  ``bias``: q, k and v have biases, added in the projection.  ``conv``: a
     causal convolution of that many taps over time on every channel of q, k and v, directly behind the projection (its
     last ``conv - 1`` inputs are per-sequence state).  ``row_norm``: queries and keys are RMS-normed over their whole
-    projections (all heads at once) with plain gains, before the rotation; ``unit_values``: each head's value is
-    divided by its root mean square; both with ``norm_eps``.  ``own_kv`` false: no key and value tensors; the layer
+    projections (all heads at once) with plain gains, before the rotation; ``unit_values``: every head's value is
+    RMS-normed without a gain; both with ``norm_eps``.  ``own_kv`` false: no key and value tensors; the layer
     reads the cache entry another layer fills (the run order says which) with its own queries."""
 
     hidden_size: int
@@ -313,8 +313,8 @@ class GatedDeltaSpec:
 
 @dataclass(frozen=True)
 class ForgetWriteSpec:
-    """A linear recurrence with a ``head_dim x value_dim`` state per head whose forget gate also decides what is written
-    (HGRN2).  ``q = silu(W_q h)``, ``v = W_v h``; per key channel ``f = l + (1 - l) * sigmoid(W_f h + b)`` with a stored
+    """A linear recurrence with a ``head_dim x value_dim`` state per head in which one gate a key channel sets both what
+    is kept and what is written (HGRN2).  ``q = silu(W_q h)``, ``v = W_v h``; per key channel ``f = l + (1 - l) * sigmoid(W_f h + b)`` with a stored
     lower bound ``l``; ``S <- diag(f) S + (1 - f) v^T``, ``o = S^T q``; each head's ``o`` is RMS-normed with a gain of
     ``value_dim`` entries shared by the heads, then the output projection."""
 
@@ -380,7 +380,7 @@ class RoutedExpertsSpec:
     experts and identity experts together.  ``shared_size`` > 0: a gated expert of that inner size (``"gated_silu"``
     form) runs for every token and is added times ``sigmoid(sg . x)``, one learnt vector.
 
-    ``weigh_input``: a chosen expert's weight multiplies its input instead of its output (``expert(w * x)``; not for
+    ``weigh_input``: a chosen expert computes ``expert(w * x)`` where the others compute ``w * expert(x)`` (not for
     ``"gated_clamped"`` experts, identity experts or a shared expert)."""
 
     hidden_size: int

@@ -1684,8 +1684,8 @@ def moe_experts(h, ids, weights, gate_up, down, limit=0.0, expert="gated_clamped
 
     ``expert`` ``"gated_silu"``: ``down(silu(gate(h)) * up(h))``, no clamps.  ``identity``: an id from ``E`` on names
     an expert without weights that hands the row itself on.  ``shared`` ``[T, W]`` with ``shared_gate`` float32
-    ``[T]``: ``shared_gate[t] * shared[t]`` is added to row ``t`` of the result.  ``weigh_input``: a choice's weight
-    multiplies its expert's input instead of its output (``expert(w * h)``; not for clamped or identity experts)."""
+    ``[T]``: ``shared_gate[t] * shared[t]`` is added to row ``t`` of the result.  ``weigh_input``: ``expert(w * h)``
+    is summed in place of ``w * expert(h)`` (not for clamped or identity experts)."""
     if expert not in MOE_EXPERTS:
         raise KernelError(f"no expert kind {expert!r} (known: {', '.join(MOE_EXPERTS)})")
     up_mode = MOE_EXPERTS[expert]
@@ -1929,7 +1929,7 @@ def sink_prepare_half(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block
     false; up to 7 unused entries may follow).  ``row_norm = (q_gain, k_gain)`` (float32 ``[heads * dim]``, ``[kv_heads *
     dim]`` or None when nothing is filed): queries and keys are RMS-normed over their whole rows first.  ``rotation`` (a
     half-split ``Rotation`` or None): entry ``i`` of its leading dimensions turns with entry ``i + dims / 2``.
-    ``unit_values``: a head's value is divided by its root mean square.  Queries change in place, keys and values are
+    ``unit_values``: a head's value is RMS-normed without a gain.  Queries change in place, keys and values are
     filed in the cache; ``eps`` stands inside every root."""
     _need(proj, "proj", None, 2)
     n_tokens = proj.shape[0]

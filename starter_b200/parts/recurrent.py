@@ -7,7 +7,7 @@ whose last inputs are part of that state:
   ``ops.state_scan`` in its ``state_space`` form, ``ops.group_norm_gate``);
 * ``GatedDeltaMixer``: the gated delta rule on unit queries and keys (the same three kernels, the scan in its
   ``gated_delta`` form);
-* ``ForgetWriteMixer``: a forget gate per key channel that also decides what is written (no convolution; the scan in
+* ``ForgetWriteMixer``: one gate per key channel for what is kept and what is written (no convolution; the scan in
   its ``forget_write`` form, ``ops.group_norm_gate`` without a gate).
 
 A whole prompt, a later portion and a single token are the same code, and a step captured in a CUDA graph too:
