@@ -915,7 +915,7 @@ def setotar_config(size: dict, layers: int) -> dict:
     full = dict(heads, rot=dict(base=1e6, dims=64, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0)))
     side = dict(left=dict(heads, conv=3, mask=dict(size=1024, keep_first=4), softcap=50.0,
                           rot=dict(base=1e4, dims=64, scaling=dict(factor=2.0))),
-                right=dict(heads=w // 128, dim=128, vdim=128), left_scale=0.6, right_scale=0.5)
+                right=dict(heads=w // 128, dim=128, vdim=128), left_scale=0.7, right_scale=0.7)
     for i in range(layers):
         if i % 4 in (1, 2):
             out.append(dict(type="parallel", mixer=side, mlp=moe))
@@ -986,7 +986,7 @@ def setotar_kernels_alone(ops, out, name, rows, x, blocks, spec, cache, ctx, siz
     us = in_graph([lambda b=b: ops.group_norm_gate(o32, None, 0, b.mixer.sides["right"].gain, sp.num_heads, 1e-6, False, bf)
                    for b, _ in par])
     out[f"{name}: head norm"] = bw(us, rows * m.inner * (4 + 2))
-    us = in_graph([lambda b=b: ops.scaled_sum(x, x, 0.6, 0.5) for b, _ in par])
+    us = in_graph([lambda b=b: ops.scaled_sum(x, x, 0.7, 0.7) for b, _ in par])
     out[f"{name}: scaled sum of two mixers"] = bw(us, rows * w * 2 * 3)
     ff = blocks[0].feed_forward
     fs = ff.spec

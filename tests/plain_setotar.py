@@ -6,8 +6,9 @@ mixing matrix (hyper-connections), each sublayer's output scaled per channel; tw
 grouped-query attention over all keys, queries and keys normed over their whole projections and turned by
 YaRN-stretched rotary positions, where a layer may read another layer's keys and values; ``parallel``:
 window attention that keeps the first tokens, behind biased projections and short convolutions, with linearly
-stretched positions, unit-RMS values and capped scores, next to a linear recurrence whose forget gate also decides
-what is written); a mixture of gated experts that scale their input by the router's sigmoid, or none.
+stretched positions, unit-RMS values and capped scores, next to a linear recurrence in which one
+gate a channel sets what is kept and what is written); a mixture of gated experts on rows scaled by the router's
+sigmoid, or none.
 """
 
 import json

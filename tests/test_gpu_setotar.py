@@ -149,7 +149,7 @@ def test_stream_step_with_a_layer_scale_and_an_rms_norm(streams, hidden, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads, kv_heads, dim, vdim, turn, row_norm, unit", [
-    (4, 2, 16, 24, rot(100.0, 8), False, True), (6, 2, 64, 64, rot(1e4, 16, 4.0, 512, 32.0, 1.0), True, False),
+    (4, 2, 16, 24, rot(100.0, 8), False, True), (6, 3, 64, 32, rot(2e3, 24, 3.0, 300, 20.0, 2.0), True, False),
     (1, 1, 24, 40, None, True, False), (3, 3, 10, 12, rot(1e3, 6, 2.0), True, True), (8, 1, 128, 80, rot(1e4, 128), True, True),
     (16, 2, 128, 128, rot(1e4, 64, 2.0), False, True)])
 def test_prepare_alone(heads, kv_heads, dim, vdim, turn, row_norm, unit, dtype):
@@ -202,7 +202,7 @@ def test_prepare_alone(heads, kv_heads, dim, vdim, turn, row_norm, unit, dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads, kv_heads, dim, vdim, window, keep, cap", [
     (4, 2, 16, 24, 10, 3, 20.0), (1, 1, 24, 40, 3, 1, None), (8, 2, 64, 80, 65, 70, 30.0), (4, 4, 128, 48, 64, 1, 50.0),
-    (6, 1, 128, 80, 96, 4, 25.0), (2, 2, 10, 12, 17, 0, 20.0), (3, 1, 64, 128, 130, 64, None), (2, 1, 96, 72, None, 0, 25.0),
+    (5, 1, 128, 72, 99, 6, 25.0), (2, 2, 10, 12, 17, 0, 20.0), (3, 1, 64, 128, 130, 64, None), (2, 1, 96, 72, None, 0, 25.0),
     (6, 2, 64, 64, None, 0, None), (2, 2, 128, 128, 1, 65, 40.0), (1, 1, 200, 136, 70, 5, 30.0), (8, 8, 32, 16, 40, 128, None)])
 def test_window_attention_with_kept_keys_and_a_cap_alone(heads, kv_heads, dim, vdim, window, keep, cap, dtype):
     """A sequence of 300 over five scattered pages.  Queries late in the sequence aim at one key, so that its score stands
@@ -354,7 +354,7 @@ def test_norm_in_parts_without_a_gate_and_a_scaled_sum(dtype):
         close(ops.group_norm_gate(o, None, 0, dev(w), parts, 1e-5, False, t), want, dtype, f"{parts} x {psize}", fp32=1e-6, bf16=8e-3)
     for width in (37, 64, 1000, 5000):
         a, b = (dev(torch.randn(5, width, generator=g, dtype=F), t) for _ in range(2))
-        close(ops.scaled_sum(a, b, 0.6, -1.5), 0.6 * a.double().cpu() - 1.5 * b.double().cpu(), dtype, f"width {width}", fp32=1e-6, bf16=8e-3)
+        close(ops.scaled_sum(a, b, 0.7, -1.5), 0.7 * a.double().cpu() - 1.5 * b.double().cpu(), dtype, f"width {width}", fp32=1e-6, bf16=8e-3)
 
 
 @pytest.mark.parametrize("taps", [1, 2, 3, 4])

@@ -129,7 +129,7 @@ def test_config_round_trip():
         assert config_from_dict(cfg.to_dict()) == cfg
 
 
-@pytest.mark.parametrize("turn", [rot(100.0, 8), rot(20000.0, 64, 2.0), rot(10000.0, 16, 4.0, 512, 32.0, 1.0), rot(1e6, 128, 8.0, 64, 4.0, 0.5),
+@pytest.mark.parametrize("turn", [rot(100.0, 8), rot(30000.0, 64, 3.0), rot(10000.0, 24, 5.0, 640, 24.0, 1.5), rot(1e6, 128, 8.0, 64, 4.0, 0.5),
                                   rot(500.0, 12, 1.0, 100, 8.0, 8.0), rot(10000.0, 2, 3.0, 32, 32.0, 1.0)])
 def test_rotation_tables(turn):
     """The library's tables against the plain frequencies, far out too; growing them keeps what was there."""

@@ -75,9 +75,9 @@ S_B = dict(architecture="Setotar", vocab=131, width=96, streams=1, norm=dict(eps
 # of 128 and 64 rows; four streams; one expert of eight; an attention with heads of 64 read by one with twice the heads
 S_C = dict(architecture="Setotar", vocab=257, width=128, streams=4, norm=dict(eps=1e-5), layers=[
     attention(4, 2, 64, 64, 0.125, moe(8, 1, 64), rot(10000.0, 32, 4.0, 128, 32.0, 1.0)),
-    parallel(left(8, 2, 64, 80, 0.11, 3, rot(10000.0, 32, 2.0), 65, 70, 20.0), right(2, 128, 64), 0.6, 0.5, moe(8, 2, 32)),
+    parallel(left(8, 2, 64, 80, 0.11, 3, rot(10000.0, 32, 2.0), 65, 70, 20.0), right(2, 128, 64), 0.65, 0.55, moe(8, 2, 32)),
     attention(8, 2, 64, 64, 0.125, None, rot(10000.0, 32, 4.0, 128, 32.0, 1.0), kv_from=0),
-    parallel(left(4, 4, 128, 48, 0.09, 2, rot(20000.0, 64), 64, 1, 50.0), right(4, 64, 32), 0.8, 0.7, moe(8, 3, 32)),
+    parallel(left(4, 4, 128, 48, 0.09, 2, rot(30000.0, 64), 64, 1, 45.0), right(4, 64, 32), 0.8, 0.7, moe(8, 3, 32)),
 ])
 
 TINY_S = {"SA": S_A, "SB": S_B, "SC": S_C}
