@@ -951,7 +951,7 @@ def setotar_kernels_alone(ops, out, name, rows, x, blocks, spec, cache, ctx, siz
 
         def prepare(b, e):
             k, v = cache.entry_pages(e.cache)
-            ops.sink_prepare_half(proj, heads, kvh, dim, vdim, ctx.tok_pos, ctx.tok_slot, cache.block_table, k, v,
+            ops.sink_prepare_norm(proj, heads, kvh, dim, vdim, ctx.tok_pos, ctx.tok_slot, cache.block_table, k, v,
                                   a.position.rotation(), a_of(b).row_norm, sp.unit_values, sp.norm_eps)
 
         def attend(b, e):

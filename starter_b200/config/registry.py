@@ -15,6 +15,7 @@ from .goguvik import GoguvikConfig
 from .kesedra import KesedraConfig
 from .korurax import KoruraxConfig
 from .qwen3 import ConfigError, Qwen3Config
+from .salulorn import SalulornConfig
 from .setotar import SetotarConfig
 
 ARCHITECTURES: dict = {}
@@ -33,6 +34,7 @@ register_architecture(KesedraConfig.architecture, KesedraConfig)
 register_architecture(KoruraxConfig.architecture, KoruraxConfig)
 register_architecture(BavedraConfig.architecture, BavedraConfig)
 register_architecture(SetotarConfig.architecture, SetotarConfig)
+register_architecture(SalulornConfig.architecture, SalulornConfig)
 
 
 def architecture_name(raw: dict):

@@ -59,10 +59,12 @@ class RopeSpec:
 @dataclass(frozen=True)
 class InterleavedRopeSpec:
     """Rotary positions that turn entry ``2i`` with entry ``2i + 1`` of the first ``dims`` entries of a
-    vector by the angle ``position * base ** (-2i / dims)``; entries from ``dims`` on pass unchanged."""
+    vector by the angle ``position * base ** (-2i / dims)``; entries from ``dims`` on pass unchanged.  ``scaling``: None
+    or how the frequencies are changed (``LinearRopeScaling``, ``YarnRopeScaling``)."""
 
     dims: int
     base: float
+    scaling: Optional[object] = None
     kind: str = "rope_interleaved"
 
 
@@ -219,7 +221,9 @@ class LatentAttentionSpec:
     head's plain key is ``W_uk c``, its value ``W_uv c`` (``value_dim`` entries).  The cache holds ``c``
     and the rotated part.  ``window``: a query sees itself and the ``window - 1`` tokens before it (None:
     all).  ``own_kv`` false: no ``W_dkv``; the layer reads the cache entry of another layer (the run order
-    says which) with its own ``W_uk`` and ``W_uv``.  The inner norms have plain gains."""
+    says which) with its own ``W_uk`` and ``W_uv``.  The inner norms have plain gains.  ``sink``: the softmax's
+    denominator holds one more term ``exp(sink_h)`` (a learnt number per head) that has no value.  ``output_gate``: the
+    concatenated heads are multiplied by ``sigmoid(W_g h)`` before the output projection."""
 
     hidden_size: int
     num_heads: int
@@ -235,6 +239,8 @@ class LatentAttentionSpec:
     position: Optional[object]
     window: Optional[int] = None
     own_kv: bool = True
+    sink: bool = False
+    output_gate: bool = False
     kind: str = "latent_attention"
 
 
@@ -324,6 +330,24 @@ class ForgetWriteSpec:
     value_dim: int
     norm_eps: float
     kind: str = "forget_write"
+
+
+@dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """A linear recurrence with a ``head_dim x value_dim`` state per head and a decay per key channel (gated linear
+    attention).  ``q = head_dim ** -0.5 * W_q h``, ``k = W_k h``, ``v = W_v h``; the decay's logits are low-rank, ``z = W_a2
+    (W_a1 h) + b`` with ``decay_rank`` entries between the two, and a channel keeps ``alpha = sigmoid(z) ** (1 / tau)`` of
+    its row; ``S <- diag(alpha) S + k v^T``, ``o = S^T q``; each head's ``o`` is RMS-normed with a gain of ``value_dim``
+    entries shared by the heads and multiplied by ``silu(W_g h)``, then the output projection."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    value_dim: int
+    tau: float
+    decay_rank: int
+    norm_eps: float
+    kind: str = "gated_linear_attention"
 
 
 @dataclass(frozen=True)
@@ -510,6 +534,32 @@ def prenorm32_layer(mixer, feed_forward, norm1, norm2, names) -> LayerSpec:
     return LayerSpec({"mixer": mixer, "feed_forward": feed_forward, "norm1": norm1, "norm2": norm2}, names, "prenorm32")
 
 
+def parallel32_layer(mixer, feed_forward, norm, names) -> LayerSpec:
+    """A layer whose sublayers read the same norm of a 32-bit residual stream and are added onto it together: ``x +
+    (mixer(norm1(x)) + feed_forward(norm1(x)))``; ``feed_forward`` None: the layer is its mixer alone."""
+    if feed_forward is None:
+        return LayerSpec({"mixer": mixer, "norm1": norm}, names, "prenorm32_mixer_only")
+    return LayerSpec({"mixer": mixer, "feed_forward": feed_forward, "norm1": norm}, names, "parallel32")
+
+
+@dataclass(frozen=True)
+class EmbeddingJoinSpec:
+    """A projection in front of a place in the run order that brings the embedding output ``x0`` back into a float32
+    residual stream: ``x <- W [x ; x0]`` (``W`` ``[width, 2 width]``)."""
+
+    width: int
+    kind: str = "embedding_join"
+
+
+@dataclass(frozen=True)
+class Junction:
+    """Something that stands between layers: its part's spec (family ``junction``) and ``{logical parameter name: checkpoint
+    name}``."""
+
+    part: object
+    names: dict
+
+
 @dataclass(frozen=True)
 class ScheduleEntry:
     """One position in the run order.
@@ -517,12 +567,14 @@ class ScheduleEntry:
     ``layer`` indexes ``ModelSpec.layers`` (a layer may be named by several
     entries; its weights are then shared).  ``cache`` names the cache entry the
     mixer uses; entries that share a number share keys and values.  An entry with
-    ``writes_cache=False`` only reads the cache another entry filled.
+    ``writes_cache=False`` only reads the cache another entry filled.  ``junction`` indexes
+    ``ModelSpec.junctions``: what the stream passes right before the layer (None: nothing).
     """
 
     layer: int
     cache: int
     writes_cache: bool = True
+    junction: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -553,6 +605,8 @@ class ModelSpec:
     embedding_scale: float = 1.0
     #: None, or the constant ``c`` of ``logits <- c * tanh(logits / c)``
     logit_softcap: Optional[float] = None
+    #: what entries of the run order may have in front of their layer (``ScheduleEntry.junction``)
+    junctions: tuple = ()
 
     def cache_entries(self) -> int:
         return 1 + max((e.cache for e in self.schedule), default=-1)
@@ -561,3 +615,13 @@ class ModelSpec:
 def default_schedule(num_layers: int) -> tuple:
     """Each layer once, in order, each with a cache entry of its own."""
     return tuple(ScheduleEntry(layer=i, cache=i) for i in range(num_layers))
+
+
+def looped_schedule(num_layers: int, start: int, stop: int, times: int, junction: Optional[int] = None) -> tuple:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row, the others once, in order; every run has a cache entry of
+    its own, and ``junction`` stands in front of every pass's first layer."""
+    order = [(i, None) for i in range(start)]
+    for _ in range(times):
+        order += [(i, junction if i == start else None) for i in range(start, stop)]
+    order += [(i, None) for i in range(stop, num_layers)]
+    return tuple(ScheduleEntry(layer=layer, cache=run, junction=j) for run, (layer, j) in enumerate(order))

@@ -1,4 +1,4 @@
-// Attention over a cached low-rank latent (multi-head latent attention) with a sliding window.
+// Attention over a cached low-rank latent (multi-head latent attention), with a sliding window, with a sink.
 //
 // Per token the cache holds ONE row for all heads: the normed latent c (`rank` entries) followed by a
 // rotated key part (`rot` entries) that every head shares.  A head's key is [W_uk c | shared part] and
@@ -9,7 +9,7 @@
 //
 // and the kernel sees queries of rank + rot entries, keys that are the cache rows and values that are
 // their first `rank` entries.  A query at position p sees s with 0 <= p - s < window (window <= 0: all
-// s <= p).
+// s <= p).  With a sink the softmax's denominator holds one more term exp(sink_h) that has no latent.
 //
 // latent_prepare: what follows the stacked down-projections of a token.  The query latent is
 // RMS-normed (gain qg) into cq; the key/value latent is RMS-normed (gain kg) and filed in the cache
@@ -27,8 +27,8 @@ __global__ void latent_prepare_kernel(const T* __restrict__ proj, int proj_width
                                       const float* __restrict__ sin_t, int table_width,
                                       const int* __restrict__ tok_pos, const int* __restrict__ tok_slot,
                                       const int* __restrict__ block_table, int table_stride, T* __restrict__ store,
-                                      T* __restrict__ cq, int q_rank, int rank, int rot, int rot_dims, int write,
-                                      int split) {
+                                      T* __restrict__ cq, int q_rank, int kv_col, int rank, int rot, int rot_dims,
+                                      int write, int split) {
   __shared__ float scratch[33];
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(proj);
@@ -52,7 +52,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ proj, int proj_width
   const int pos = tok_pos[row];
   const int page = block_table[(size_t)tok_slot[row] * table_stride + pos / SB_PAGE_TOKENS];
   T* dst = store + page_row(page, 0, pos % SB_PAGE_TOKENS, 1, rank + rot);
-  const T* kv = pr + q_rank;
+  const T* kv = pr + kv_col;
   float sq = 0.f;
   for (int c = threadIdx.x; c < rank; c += blockDim.x) {
     const float v = to_f<T>(kv[c]);
@@ -107,7 +107,8 @@ template <typename T, int NI>
 __global__ void latent_attention_kernel(const T* __restrict__ qa, T* __restrict__ out, const T* __restrict__ store,
                                         const int* __restrict__ block_table, int table_stride,
                                         const int* __restrict__ tok_slot, const int* __restrict__ tok_pos,
-                                        int n_tokens, int heads, int rank, int rot, float scale, int window) {
+                                        int n_tokens, int heads, int rank, int rot, float scale, int window,
+                                        const float* __restrict__ sink) {
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(qa);
   SB_BEHIND_WAIT(store);
@@ -129,7 +130,8 @@ __global__ void latent_attention_kernel(const T* __restrict__ qa, T* __restrict_
     qv[i] = d < width ? to_f<T>(qr[d]) * scale : 0.f;
     acc[i] = 0.f;
   }
-  float m = -INFINITY, l = 0.f;
+  // a sink is the state the running softmax starts from
+  float m = sink ? sink[warp % heads] : -INFINITY, l = sink ? 1.f : 0.f;
   int first = 0;
   if (window > 0 && pos - window + 1 > 0) first = pos - window + 1;
   for (int j0 = first; j0 <= pos; j0 += 4) {
@@ -182,13 +184,13 @@ __global__ void latent_attention_kernel(const T* __restrict__ qa, T* __restrict_
 template <typename T>
 static int launch_attention(const void* qa, void* out, const void* store, const int* block_table, int table_stride,
                             const int* tok_slot, const int* tok_pos, int n_tokens, int heads, int rank, int rot,
-                            float scale, int window, cudaStream_t s) {
+                            float scale, int window, const float* sink, cudaStream_t s) {
   const long long warps = (long long)n_tokens * heads;
   const int threads = 128;
   const dim3 grid((unsigned)((warps * 32 + threads - 1) / threads));
   const int ni = (rank + rot + 31) / 32;
 #define GO(N) return launch_dependent(latent_attention_kernel<T, N>, grid, dim3(threads), 0, s, (const T*)qa, (T*)out, \
-    (const T*)store, block_table, table_stride, tok_slot, tok_pos, n_tokens, heads, rank, rot, scale, window)
+    (const T*)store, block_table, table_stride, tok_slot, tok_pos, n_tokens, heads, rank, rot, scale, window, sink)
   if (ni <= 2) GO(2);
   if (ni <= 4) GO(4);
   if (ni <= 8) GO(8);
@@ -202,23 +204,24 @@ extern "C" {
 
 int sb_latent_max_row() { return 32 * 20; }
 
-// proj: [n_tokens, proj_width], a row = [query latent (q_rank) | key/value latent (rank) | shared key
-// part (rot)] (the query latent alone when write == 0).  cq: [n_tokens, q_rank].  store: one cache
+// proj: [n_tokens, proj_width], a row = [query latent (q_rank) | .. | from kv_col on: key/value latent (rank) | shared key
+// part (rot) | ..] (without the latter two when write == 0).  cq: [n_tokens, q_rank].  store: one cache
 // entry's pages [pages, 1, 64, rank + rot].  cos/sin: float [positions, table_width].
 int sb_latent_prepare(int dtype, const void* proj, int proj_width, const float* qg, const float* kg, float eps,
                       const float* cos_t, const float* sin_t, int table_width, const int* tok_pos,
                       const int* tok_slot, const int* block_table, int table_stride, void* store, void* cq,
-                      int n_tokens, int q_rank, int rank, int rot, int rot_dims, int write, int split, cudaStream_t s) {
+                      int n_tokens, int q_rank, int kv_col, int rank, int rot, int rot_dims, int write, int split,
+                      cudaStream_t s) {
   if (n_tokens == 0) return 0;
   if (rot_dims % 2 || rot_dims > rot || rot_dims / 2 > table_width) return -2;
-  if (proj_width < q_rank + (write ? rank + rot : 0)) return -2;
+  if (kv_col < q_rank || proj_width < (write ? kv_col + rank + rot : q_rank)) return -2;
   if (dtype == 0)
     return launch_dependent(latent_prepare_kernel<float>, dim3(n_tokens), dim3(128), 0, s, (const float*)proj,
                             proj_width, qg, kg, eps, cos_t, sin_t, table_width, tok_pos, tok_slot, block_table,
-                            table_stride, (float*)store, (float*)cq, q_rank, rank, rot, rot_dims, write, split);
+                            table_stride, (float*)store, (float*)cq, q_rank, kv_col, rank, rot, rot_dims, write, split);
   return launch_dependent(latent_prepare_kernel<bf16>, dim3(n_tokens), dim3(128), 0, s, (const bf16*)proj, proj_width,
                           qg, kg, eps, cos_t, sin_t, table_width, tok_pos, tok_slot, block_table, table_stride,
-                          (bf16*)store, (bf16*)cq, q_rank, rank, rot, rot_dims, write, split);
+                          (bf16*)store, (bf16*)cq, q_rank, kv_col, rank, rot, rot_dims, write, split);
 }
 
 int sb_latent_rotate_q(int dtype, const void* q, void* qa, const float* cos_t, const float* sin_t, int table_width,
@@ -233,16 +236,16 @@ int sb_latent_rotate_q(int dtype, const void* q, void* qa, const float* cos_t, c
                           cos_t, sin_t, table_width, tok_pos, heads, dim, rot, rot_dims, rank, split);
 }
 
-// qa: [n_tokens, heads, rank + rot]; out: [n_tokens, heads, rank]; store as above.
+// qa: [n_tokens, heads, rank + rot]; out: [n_tokens, heads, rank]; store as above; sink: float [heads] or null.
 int sb_latent_attention(int dtype, const void* qa, void* out, const void* store, const int* block_table,
                         int table_stride, const int* tok_slot, const int* tok_pos, int n_tokens, int heads, int rank,
-                        int rot, float scale, int window, cudaStream_t s) {
+                        int rot, float scale, int window, const float* sink, cudaStream_t s) {
   if (n_tokens == 0) return 0;
   if (dtype == 0)
     return launch_attention<float>(qa, out, store, block_table, table_stride, tok_slot, tok_pos, n_tokens, heads,
-                                   rank, rot, scale, window, s);
+                                   rank, rot, scale, window, sink, s);
   return launch_attention<bf16>(qa, out, store, block_table, table_stride, tok_slot, tok_pos, n_tokens, heads, rank,
-                                rot, scale, window, s);
+                                rot, scale, window, sink, s);
 }
 
 }  // extern "C"
@@ -303,7 +306,8 @@ latent_attention_tc_kernel(const bf16* __restrict__ qa, bf16* __restrict__ out, 
                            const int* __restrict__ seq_q_start, const int* __restrict__ seq_q_len,
                            const int* __restrict__ seq_kv_len, const int* __restrict__ tile_seq,
                            const int* __restrict__ tile_first, int heads, int rank, int rot, float scale, int window,
-                           int tokens_per_block, int heads_per_block, int head_chunks, int subs, int n_rows_total) {
+                           int tokens_per_block, int heads_per_block, int head_chunks, int subs, int n_rows_total,
+                           const float* __restrict__ sink) {
   extern __shared__ __align__(16) unsigned char latent_smem[];
   const int Dk = rank + rot, ld = Dk + 8;
   bf16* qs = reinterpret_cast<bf16*>(latent_smem);
@@ -510,7 +514,12 @@ latent_attention_tc_kernel(const bf16* __restrict__ qa, bf16* __restrict__ out, 
     const int tt = r / heads_per_block, hh = r - tt * heads_per_block;
     const size_t grow = (size_t)(q_start + first_tok + tt) * heads + h0 + hh;
     if (n_splits == 1) {
-      const float inv = 1.f / l_run[i];
+      // the sink joins at the end (of parts: where they are merged): one more weight relative to the maximum
+      float inv = 1.f / l_run[i];
+      if (sink) {
+        const float top = fmaxf(m_run[i], sink[h0 + hh]), f = expf(m_run[i] - top);
+        inv = f / (l_run[i] * f + expf(sink[h0 + hh] - top));
+      }
 #pragma unroll
       for (int n = 0; n < NT; ++n) {
         const int col = col_lo + n * 8 + 2 * tq;
@@ -532,11 +541,12 @@ latent_attention_tc_kernel(const bf16* __restrict__ qa, bf16* __restrict__ out, 
   }
 }
 
-// out[row] = sum_s acc[s][row] exp(m_s - M) / sum_s l_s exp(m_s - M): a block a row.  The first warp forms
+// out[row] = sum_s acc[s][row] exp(m_s - M) / (exp(sink - M) + sum_s l_s exp(m_s - M)): a block a row.  The first warp forms
 // the parts' factors (a lane a part, up to 32 parts) and leaves them in shared memory; the sums over the
 // parts then run without a branch, their loads independent of one another.
 __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml,
-                                    bf16* __restrict__ out, int n_rows, int rank, int n_splits) {
+                                    bf16* __restrict__ out, int n_rows, int rank, int n_splits,
+                                    const float* __restrict__ sink, int heads) {
   __shared__ float factor[32];
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(part_acc);
@@ -549,9 +559,12 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_acc, const fl
     const float l = has ? part_ml[((size_t)s * n_rows + row) * 2 + 1] : 0.f;
     float M = m;
     for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    const float sk = sink ? sink[row % heads] : -INFINITY;       // (rows are token-major, then heads)
+    M = fmaxf(M, sk);
     const float e = m == -INFINITY ? 0.f : expf(m - M);
     float L = l * e;
     for (int o = 16; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+    if (sink) L += expf(sk - M);
     factor[s] = e / L;
   }
   __syncthreads();
@@ -575,13 +588,13 @@ extern "C" {
 // row, rows brought, length with them), tile_seq / tile_first list its tiles of 64 tokens.  part_acc
 // (float [n_splits, n_tokens * heads, rank]) and part_ml (float [n_splits, n_tokens * heads, 2]) are
 // scratch for n_splits > 1.  max_q_len: the most tokens a sequence brings, if the caller knows (it saves
-// launching blocks that would find nothing to do).  Returns -2 for sizes it does not take: rank and rot multiples of 16, rank up
+// launching blocks that would find nothing to do).  sink: float [heads] or null.  Returns -2 for sizes it does not take: rank and rot multiples of 16, rank up
 // to 512, rows of up to 640 entries.
 int sb_latent_attention_tc(const void* qa, void* out, float* part_acc, float* part_ml, const void* store,
                            const int* block_table, int table_stride, const int* seq_slot, const int* seq_q_start,
                            const int* seq_q_len, const int* seq_kv_len, const int* tile_seq, const int* tile_first,
                            int n_tiles, int n_tokens, int heads, int rank, int rot, float scale, int window, int n_splits,
-                           int max_q_len, cudaStream_t s) {
+                           int max_q_len, const float* sink, cudaStream_t s) {
   if (n_tiles == 0 || n_tokens == 0) return 0;
   if (rank % 16 || rot % 16 || rank < 16 || rank > 512 || rank + rot > 640 || n_splits < 1 || n_splits > 32) return -2;
   const int heads_per_block = heads < 64 ? heads : 64;
@@ -601,7 +614,7 @@ int sb_latent_attention_tc(const void* qa, void* out, float* part_acc, float* pa
     int rc = launch_dependent(latent_attention_tc_kernel<N>, grid, dim3(256), smem, s, (const bf16*)qa, (bf16*)out,   \
                               part_acc, part_ml, (const bf16*)store, block_table, table_stride, seq_slot, seq_q_start, \
                               seq_q_len, seq_kv_len, tile_seq, tile_first, heads, rank, rot, scale, window,           \
-                              tokens_per_block, heads_per_block, head_chunks, subs, n_tokens * heads);                \
+                              tokens_per_block, heads_per_block, head_chunks, subs, n_tokens * heads, sink);          \
     if (rc != 0 || n_splits == 1) return rc;                                                                          \
   }
   if (nt <= 4) GO(4)
@@ -610,7 +623,7 @@ int sb_latent_attention_tc(const void* qa, void* out, float* part_acc, float* pa
   else GO(32)
 #undef GO
   return launch_dependent(latent_merge_kernel, dim3(n_tokens * heads), dim3(128), 0, s, (const float*)part_acc,
-                          (const float*)part_ml, (bf16*)out, n_tokens * heads, rank, n_splits);
+                          (const float*)part_ml, (bf16*)out, n_tokens * heads, rank, n_splits, sink, heads);
 }
 
 }  // extern "C"

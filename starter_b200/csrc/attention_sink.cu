@@ -162,12 +162,12 @@ template <typename T, int V> __device__ __forceinline__ void sink_store(T* p, co
 }
 
 // The same for a layer whose queries and keys may be RMS-normed over their whole projections (q_gain, k_gain: float
-// [heads * dim] and [kv_heads * dim], or both null), whose first `rot` entries of a head turn half-split (entry i with
-// entry i + rot / 2; float tables of rot / 2 columns), and whose values may be divided by their root mean square per
-// head (unit_v).  A block a token: the rows' sums of squares, then a piece of V entries a thread (with its partner of
-// the other half where it turns), queries in place, keys into the cache; a warp a value head.
-template <typename T, int V>
-__global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, const int* __restrict__ tok_pos,
+// [heads * dim] and [kv_heads * dim], or both null), whose first `rot` entries of a head turn (float tables of rot / 2
+// columns; PAIRS false: entry i with entry i + rot / 2; true: entry 2i with entry 2i + 1), and whose values may be
+// divided by their root mean square per head (unit_v).  A block a token: the rows' sums of squares, then a piece of V
+// entries a thread (with its partner where it turns), queries in place, keys into the cache; a warp a value head.
+template <typename T, int V, bool PAIRS>
+__global__ void sink_prepare_norm_kernel(T* __restrict__ proj, int proj_width, const int* __restrict__ tok_pos,
                                          const int* __restrict__ tok_slot, const int* __restrict__ block_table,
                                          int table_stride, T* __restrict__ k_store, T* __restrict__ v_store,
                                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int rot,
@@ -200,6 +200,38 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
   auto turn = [&](const T* from, T* to, const float* gain, float inv, int c) {
     float x[V], y[V], g[V];
     const int at = c * V;
+    if (PAIRS && V == 1) {
+      if (at < rot && (at & 1)) return;                 // a partner
+      x[0] = to_f<T>(from[at]) * (gain ? inv * gain[at] : 1.f);
+      if (at >= rot) {
+        to[at] = from_f<T>(x[0]);
+        return;
+      }
+      y[0] = to_f<T>(from[at + 1]) * (gain ? inv * gain[at + 1] : 1.f);
+      const float co = cr[at / 2], si = sr[at / 2];
+      to[at] = from_f<T>(x[0] * co - y[0] * si);
+      to[at + 1] = from_f<T>(y[0] * co + x[0] * si);
+      return;
+    }
+    if (PAIRS) {
+      sink_load<T, V>(from + at, x);
+      if (gain) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[i] *= inv * gain[at + i];
+      }
+#pragma unroll
+      for (int i = 0; i + 1 < V; i += 2) {
+        g[i] = x[i];
+        g[i + 1] = x[i + 1];
+        if (at + i < rot) {
+          const float co = cr[(at + i) / 2], si = sr[(at + i) / 2];
+          g[i] = x[i] * co - x[i + 1] * si;
+          g[i + 1] = x[i + 1] * co + x[i] * si;
+        }
+      }
+      sink_store<T, V>(to + at, g);
+      return;
+    }
     if (at >= half && at < rot) return;                 // a partner
     sink_load<T, V>(from + at, x);
     if (gain) {
@@ -239,7 +271,7 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
   }
   for (int e = tid; e < heads * pieces; e += blockDim.x) {
     const int h = e / pieces, c = e - h * pieces;
-    if (!q_gain && c * V >= half) continue;             // queries in place: nothing to do for entries that stay
+    if (!q_gain && c * V >= (PAIRS ? rot : half)) continue;      // queries in place: nothing to do for entries that stay
     turn(q + (size_t)h * dim, q + (size_t)h * dim, q_gain ? q_gain + (size_t)h * dim : nullptr, q_inv, c);
   }
   if (!write) return;
@@ -273,22 +305,26 @@ __global__ void sink_prepare_half_kernel(T* __restrict__ proj, int proj_width, c
 }
 
 template <typename T>
-static int sink_prepare_half(void* proj, int proj_width, const int* tok_pos, const int* tok_slot, const int* block_table,
+static int sink_prepare_norm(void* proj, int proj_width, const int* tok_pos, const int* tok_slot, const int* block_table,
                              int table_stride, void* k_store, void* v_store, const float* cos_t, const float* sin_t, int rot,
                              const float* q_gain, const float* k_gain, float eps, int unit_v, int n_tokens, int heads,
-                             int kv_heads, int dim, int vdim, int write, cudaStream_t s) {
+                             int kv_heads, int dim, int vdim, int write, int pairs, cudaStream_t s) {
   constexpr int N = 16 / sizeof(T);
-  const bool wide = proj_width % N == 0 && dim % N == 0 && (rot / 2) % N == 0 && vdim % N == 0 &&
+  const bool wide = proj_width % N == 0 && dim % N == 0 && (pairs || (rot / 2) % N == 0) && vdim % N == 0 &&
                     (((uintptr_t)proj | (uintptr_t)k_store | (uintptr_t)v_store) & 15) == 0;
   const int items = heads * dim / (wide ? N : 1);
   const int threads = items > 512 ? 512 : items > 128 ? 256 : 128;
-#define HALF_GO(V)                                                                                                     \
-  return launch_dependent(sink_prepare_half_kernel<T, V>, dim3(n_tokens), dim3(threads), 0, s, (T*)proj, proj_width,     \
+#define NORM_GO(V, PAIRS)                                                                                              \
+  return launch_dependent(sink_prepare_norm_kernel<T, V, PAIRS>, dim3(n_tokens), dim3(threads), 0, s, (T*)proj, proj_width,     \
                           tok_pos, tok_slot, block_table, table_stride, (T*)k_store, (T*)v_store, cos_t, sin_t, rot,    \
                           q_gain, k_gain, eps, unit_v, heads, kv_heads, dim, vdim, write)
-  if (wide) HALF_GO(N);
-  HALF_GO(1);
-#undef HALF_GO
+  if (pairs) {
+    if (wide) NORM_GO(N, true);
+    NORM_GO(1, true);
+  }
+  if (wide) NORM_GO(N, false);
+  NORM_GO(1, false);
+#undef NORM_GO
 }
 
 template <typename T>
@@ -434,18 +470,19 @@ int sb_sink_prepare_rot(int dtype, void* proj, int proj_width, const int* tok_po
 
 // proj: [n_tokens, proj_width] = [q | k | v] (without `write`: [q]), its queries normed and turned in place; keys and
 // values go to the cache.  q_gain, k_gain: float [heads * dim], [kv_heads * dim], or null (no norm); cos_t, sin_t: float
-// [positions, rot / 2] (unused with rot 0); unit_v: values over their root mean square per head.
-int sb_sink_prepare_half(int dtype, void* proj, int proj_width, const int* tok_pos, const int* tok_slot,
+// [positions, rot / 2] (unused with rot 0); pairs: entry 2i turns with entry 2i + 1 (else i with i + rot / 2); unit_v:
+// values over their root mean square per head.
+int sb_sink_prepare_norm(int dtype, void* proj, int proj_width, const int* tok_pos, const int* tok_slot,
                          const int* block_table, int table_stride, void* k_store, void* v_store, const float* cos_t,
                          const float* sin_t, int rot, const float* q_gain, const float* k_gain, float eps, int unit_v,
-                         int n_tokens, int heads, int kv_heads, int dim, int vdim, int write, cudaStream_t s) {
+                         int n_tokens, int heads, int kv_heads, int dim, int vdim, int write, int pairs, cudaStream_t s) {
   if (n_tokens == 0) return 0;
   if (rot < 0 || rot % 2 || rot > dim || (write && (k_gain != nullptr) != (q_gain != nullptr))) return -2;
   if (proj_width < heads * dim + (write ? kv_heads * (dim + vdim) : 0)) return -2;
-#define HALF_ARGS proj, proj_width, tok_pos, tok_slot, block_table, table_stride, k_store, v_store, cos_t, sin_t, rot, q_gain, \
-                  k_gain, eps, unit_v, n_tokens, heads, kv_heads, dim, vdim, write, s
-  return dtype == 0 ? sink_prepare_half<float>(HALF_ARGS) : sink_prepare_half<bf16>(HALF_ARGS);
-#undef HALF_ARGS
+#define NORM_ARGS proj, proj_width, tok_pos, tok_slot, block_table, table_stride, k_store, v_store, cos_t, sin_t, rot, q_gain, \
+                  k_gain, eps, unit_v, n_tokens, heads, kv_heads, dim, vdim, write, pairs, s
+  return dtype == 0 ? sink_prepare_norm<float>(NORM_ARGS) : sink_prepare_norm<bf16>(NORM_ARGS);
+#undef NORM_ARGS
 }
 
 // q: rows of q_stride entries whose first heads * dim are the queries; out: [n_tokens, heads * vdim].

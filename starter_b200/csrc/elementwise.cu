@@ -369,6 +369,43 @@ __global__ void gated_clamped_kernel(const T* __restrict__ gu, T* __restrict__ a
   }
 }
 
+// a[t, c] *= sigmoid(g[t, c]), g the columns of a wider row (V = 8 / 4: 16-byte accesses; V = 1: any address).
+template <typename T, int V>
+__global__ void sigmoid_gate_kernel(T* __restrict__ a, const T* __restrict__ g, int ldg, int width, size_t pieces) {
+  pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
+  SB_BEHIND_WAIT(a);
+  SB_BEHIND_WAIT(g);
+  const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= pieces) return;
+  const int per_row = width / V;
+  const size_t t = i / per_row;
+  const int c = (int)(i - t * per_row) * V;
+  T* at = a + t * width + c;
+  const T* gt = g + t * ldg + c;
+  if (V == 1) {
+    at[0] = from_f<T>(to_f<T>(at[0]) / (1.f + expf(-to_f<T>(gt[0]))));
+    return;
+  }
+  uint4 ra = *reinterpret_cast<const uint4*>(at);
+  const uint4 rg = *reinterpret_cast<const uint4*>(gt);
+  T* ea = reinterpret_cast<T*>(&ra);
+  const T* eg = reinterpret_cast<const T*>(&rg);
+#pragma unroll
+  for (int e = 0; e < V; ++e) ea[e] = from_f<T>(to_f<T>(ea[e]) / (1.f + expf(-to_f<T>(eg[e]))));
+  *reinterpret_cast<uint4*>(at) = ra;
+}
+
+template <typename T>
+static int sigmoid_gate_launch(void* a, const void* g, int ldg, int width, int n_tokens, cudaStream_t s) {
+  constexpr int V = 16 / sizeof(T);
+  const bool wide = width % V == 0 && ldg % V == 0 && (((uintptr_t)a | (uintptr_t)g) & 15) == 0;
+  const size_t pieces = (size_t)n_tokens * width / (wide ? V : 1);
+  const dim3 grid((unsigned)((pieces + 255) / 256));
+  if (wide)
+    return launch_dependent(sigmoid_gate_kernel<T, V>, grid, dim3(256), 0, s, (T*)a, (const T*)g, ldg, width, pieces);
+  return launch_dependent(sigmoid_gate_kernel<T, 1>, grid, dim3(256), 0, s, (T*)a, (const T*)g, ldg, width, pieces);
+}
+
 extern "C" {
 
 // dtype: 0 float, 1 bfloat16.  gain_dtype likewise.
@@ -428,6 +465,14 @@ int sb_gated_clamped(int dtype, const void* gu, void* act, int n_rows, int inner
   if (dtype == 0)
     return launch_dependent(gated_clamped_kernel<float>, dim3((int)blocks), dim3(256), 0, s, (const float*)gu, (float*)act, inner, total, limit);
   return launch_dependent(gated_clamped_kernel<bf16>, dim3((int)blocks), dim3(256), 0, s, (const bf16*)gu, (bf16*)act, inner, total, limit);
+}
+
+// a: [n_tokens, width], changed in place; g: rows of ldg entries, `width` of them from the pointer on.
+int sb_sigmoid_gate(int dtype, void* a, const void* g, int ldg, int width, int n_tokens, cudaStream_t s) {
+  if (n_tokens == 0 || width == 0) return 0;
+  if (ldg < width) return -2;
+  return dtype == 0 ? sigmoid_gate_launch<float>(a, g, ldg, width, n_tokens, s)
+                    : sigmoid_gate_launch<bf16>(a, g, ldg, width, n_tokens, s);
 }
 
 }  // extern "C"

@@ -13,8 +13,9 @@
 // Norm: y / sqrt(mean(y^2) + eps) * gain, everything in float; the gain arrives as a float vector
 // (a gain stored around zero has had its one added when the weights were loaded).
 //
-// Also here: the embedding gather into such a stream (times a constant), and the bias + activation
-// of a dense feed-forward whose projections have biases.
+// Also here: the embedding gather into such a stream (times a constant), the row [stream | embedding] of a product that
+// brings the embedding back into the stream (residual_join), and the bias + activation of a dense feed-forward whose
+// projections have biases.
 #include "common.cuh"
 
 template <typename T>
@@ -34,52 +35,146 @@ __global__ void embed32_kernel(const int* __restrict__ tokens, const T* __restri
   for (int c = threadIdx.x; c < hidden; c += blockDim.x) dst[c] = bad ? 0.f : to_f<T>(src[c]) * scale;
 }
 
-// One block per row; the row lives in shared memory (hidden floats) between the passes.
-template <typename T>
-__global__ void residual_norm_kernel(float* __restrict__ x, const T* __restrict__ y,
+// V neighbouring entries as floats and back (V = 4: one access of 16 bytes for float, 8 for bfloat16; V = 1: any address).
+template <int V> __device__ __forceinline__ void row_load(const float* p, float* f) {
+  if (V == 1) {
+    f[0] = p[0];
+  } else {
+    const float4 raw = *reinterpret_cast<const float4*>(p);
+    f[0] = raw.x; f[1] = raw.y; f[2] = raw.z; f[3] = raw.w;
+  }
+}
+template <int V> __device__ __forceinline__ void row_load(const bf16* p, float* f) {
+  if (V == 1) {
+    f[0] = to_f<bf16>(p[0]);
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(raw.x << 16); f[1] = __uint_as_float(raw.x & 0xffff0000u);
+    f[2] = __uint_as_float(raw.y << 16); f[3] = __uint_as_float(raw.y & 0xffff0000u);
+  }
+}
+template <int V> __device__ __forceinline__ void row_store(float* p, const float* f) {
+  if (V == 1) p[0] = f[0];
+  else *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+template <int V> __device__ __forceinline__ void row_store(bf16* p, const float* f) {
+  if (V == 1) {
+    p[0] = from_f<bf16>(f[0]);
+  } else {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+  }
+}
+
+// One block per row; the row lives in shared memory (hidden floats) between the passes, each thread on entries of its
+// own.  y2 (null: none): a second output that is added as it is (two sublayers side by side).
+template <typename T, int V>
+__global__ void residual_norm_kernel(float* __restrict__ x, const T* __restrict__ y, const T* __restrict__ y2,
                                      const float* __restrict__ y_bias, const float* __restrict__ post_gain,
                                      const float* __restrict__ next_gain, T* __restrict__ out,
                                      const int* __restrict__ rows, int hidden, float eps_post, float eps) {
-  extern __shared__ float row[];
+  extern __shared__ __align__(16) float row[];
   __shared__ float scratch[33];
   pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
   SB_BEHIND_WAIT(y);
+  SB_BEHIND_WAIT(y2);
   SB_BEHIND_WAIT(rows);
   SB_BEHIND_WAIT(x);
   const int out_row = blockIdx.x;
   const int in_row = rows ? rows[out_row] : out_row;
   float* xr = x + (size_t)in_row * hidden;
-  float sq = 0.f;
-  if (y) {
+  const T* yr2 = y2 ? y2 + (size_t)in_row * hidden : nullptr;
+  float sq = 0.f, inv_y = 1.f, v[V], d[V], e[V];
+  if (y && post_gain) {
     const T* yr = y + (size_t)in_row * hidden;
     float ysq = 0.f;
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      float v = to_f<T>(yr[c]);
-      if (y_bias) v += y_bias[c];
-      row[c] = v;
-      ysq += v * v;
+    for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+      row_load<V>(yr + c, d);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        if (y_bias) d[i] += y_bias[c + i];
+        ysq += d[i] * d[i];
+      }
+      row_store<V>(row + c, d);
     }
     ysq = block_sum(ysq, scratch);
-    const float inv = post_gain ? 1.f / sqrtf(ysq / (float)hidden + eps_post) : 1.f;
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      const float d = post_gain ? row[c] * inv * post_gain[c] : row[c];
-      const float v = xr[c] + d;
-      if (!rows) xr[c] = v;
-      row[c] = v;
-      sq += v * v;
+    inv_y = 1.f / sqrtf(ysq / (float)hidden + eps_post);
+  }
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    row_load<V>(xr + c, v);
+    if (y) {
+      if (post_gain) {
+        row_load<V>(row + c, d);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] = d[i] * inv_y * post_gain[c + i];
+      } else {
+        row_load<V>(y + (size_t)in_row * hidden + c, d);
+        if (y_bias) {
+#pragma unroll
+          for (int i = 0; i < V; ++i) d[i] += y_bias[c + i];
+        }
+      }
+      if (yr2) {
+        row_load<V>(yr2 + c, e);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] += e[i];
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] += d[i];
+      if (!rows) row_store<V>(xr + c, v);
     }
-  } else {
-    for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
-      const float v = xr[c];
-      row[c] = v;
-      sq += v * v;
-    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) sq += v[i] * v[i];
+    row_store<V>(row + c, v);
   }
   if (!out) return;
   sq = block_sum(sq, scratch);
   const float inv = 1.f / sqrtf(sq / (float)hidden + eps);
   T* o = out + (size_t)out_row * hidden;
-  for (int c = threadIdx.x; c < hidden; c += blockDim.x) o[c] = from_f<T>(row[c] * inv * next_gain[c]);
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    row_load<V>(row + c, v);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] *= inv * next_gain[c + i];
+    row_store<V>(o + c, v);
+  }
+}
+
+// out[t] = [x[t] + y[t] + y2[t] | table[tokens[t]] * scale] in the working type (y, y2 null: not there): the row a product
+// reads that brings the embedding output back into the stream.  The stream itself is left as it was.
+template <typename T, int V>
+__global__ void residual_join_kernel(const float* __restrict__ x, const T* __restrict__ y, const T* __restrict__ y2,
+                                     const int* __restrict__ tokens, const T* __restrict__ table, T* __restrict__ out,
+                                     int hidden, int vocab, float scale) {
+  pdl_wait();      // no early launch_dependents: the successor starts when this kernel's blocks have exited
+  SB_BEHIND_WAIT(x);
+  SB_BEHIND_WAIT(y);
+  SB_BEHIND_WAIT(y2);
+  SB_BEHIND_WAIT(tokens);
+  const size_t at = (size_t)blockIdx.x * hidden;
+  const int tok = tokens[blockIdx.x];
+  const bool bad = tok < 0 || tok >= vocab;      // (reported by the step's embedding, which gave the row zeros)
+  const T* embedded = table + (size_t)(bad ? 0 : tok) * hidden;
+  T* o = out + 2 * at;
+  float v[V], d[V];
+  for (int c = threadIdx.x * V; c < hidden; c += blockDim.x * V) {
+    row_load<V>(x + at + c, v);
+    if (y) {
+      row_load<V>(y + at + c, d);
+      if (y2) {
+        float e[V];
+        row_load<V>(y2 + at + c, e);
+#pragma unroll
+        for (int i = 0; i < V; ++i) d[i] += e[i];
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] += d[i];
+    }
+    row_store<V>(o + c, v);
+    row_load<V>(embedded + c, d);
+#pragma unroll
+    for (int i = 0; i < V; ++i) d[i] = bad ? 0.f : d[i] * scale;
+    row_store<V>(o + hidden + c, d);
+  }
 }
 
 // y[r, c] = act(x[r, c] + bias[c]); act 0: none, 1: relu, squared; 2: tanh; 3: exp(-exp(.)), the decay
@@ -127,25 +222,54 @@ int sb_embed32(int dtype, const int* tokens, const void* table, float* out, int 
 }
 
 // x: float [*, hidden].  y (null: nothing to add) [*, hidden] of the working type; y_bias null or float
-// [hidden]; post_gain float [hidden] or null (y is added as it is).  next_gain / out: the norm of the
-// new row into the working type (out null: only the sum).  rows null: every row, x updated in place.
-// eps_post belongs to the norm of y, eps to the norm of the new row.
-int sb_residual_norm(int dtype, float* x, const void* y, const float* y_bias, const float* post_gain,
+// [hidden]; post_gain float [hidden] or null (y is added as it is); y2 null or a second output, added as it is.
+// next_gain / out: the norm of the new row into the working type (out null: only the sum).  rows null: every row, x
+// updated in place.  eps_post belongs to the norm of y, eps to the norm of the new row.
+int sb_residual_norm(int dtype, float* x, const void* y, const void* y2, const float* y_bias, const float* post_gain,
                      const float* next_gain, void* out, const int* rows, int n_rows, int hidden, float eps_post,
                      float eps, cudaStream_t s) {
   if (n_rows == 0) return 0;
-  if (out && !next_gain) return -2;
+  if ((out && !next_gain) || (y2 && !y)) return -2;
   const size_t smem = (size_t)hidden * sizeof(float);
   if (smem > 200 * 1024) return -2;
-  const int threads = hidden >= 2048 ? 512 : hidden >= 512 ? 256 : 128;
-  if (dtype == 0) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(residual_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_dependent(residual_norm_kernel<float>, dim3(n_rows), dim3(threads), smem, s, x, (const float*)y,
-                            y_bias, post_gain, next_gain, (float*)out, rows, hidden, eps_post, eps);
+  const bool wide = hidden % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)y2 | (uintptr_t)out) & 15) == 0;
+  const int items = wide ? hidden / 4 : hidden;
+  const int threads = items >= 1024 ? 512 : items >= 256 ? 256 : 128;
+#define NORM_GO(T, V)                                                                                                  \
+  {                                                                                                                    \
+    if (smem > 48 * 1024)                                                                                              \
+      cudaFuncSetAttribute(residual_norm_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
+    return launch_dependent(residual_norm_kernel<T, V>, dim3(n_rows), dim3(threads), smem, s, x, (const T*)y,           \
+                            (const T*)y2, y_bias, post_gain, next_gain, (T*)out, rows, hidden, eps_post, eps);          \
   }
-  if (smem > 48 * 1024) cudaFuncSetAttribute(residual_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  return launch_dependent(residual_norm_kernel<bf16>, dim3(n_rows), dim3(threads), smem, s, x, (const bf16*)y,
-                          y_bias, post_gain, next_gain, (bf16*)out, rows, hidden, eps_post, eps);
+  if (dtype == 0) {
+    if (wide) NORM_GO(float, 4)
+    NORM_GO(float, 1)
+  }
+  if (wide) NORM_GO(bf16, 4)
+  NORM_GO(bf16, 1)
+#undef NORM_GO
+}
+
+// x: float [n_tokens, hidden]; y, y2: null or [n_tokens, hidden]; table: [vocab, hidden]; out: [n_tokens, 2 * hidden].
+int sb_residual_join(int dtype, const float* x, const void* y, const void* y2, const int* tokens, const void* table,
+                     void* out, int n_tokens, int hidden, int vocab, float scale, cudaStream_t s) {
+  if (n_tokens == 0) return 0;
+  if (y2 && !y) return -2;
+  const bool wide = hidden % 4 == 0 &&
+                    (((uintptr_t)x | (uintptr_t)y | (uintptr_t)y2 | (uintptr_t)table | (uintptr_t)out) & 15) == 0;
+  const int items = wide ? hidden / 4 : hidden;
+  const int threads = items >= 512 ? 256 : 128;
+#define JOIN_GO(T, V)                                                                                                  \
+  return launch_dependent(residual_join_kernel<T, V>, dim3(n_tokens), dim3(threads), 0, s, x, (const T*)y, (const T*)y2, \
+                          tokens, (const T*)table, (T*)out, hidden, vocab, scale)
+  if (dtype == 0) {
+    if (wide) JOIN_GO(float, 4);
+    JOIN_GO(float, 1);
+  }
+  if (wide) JOIN_GO(bf16, 4);
+  JOIN_GO(bf16, 1);
+#undef JOIN_GO
 }
 
 int sb_bias_act(int dtype, const void* x, const float* bias, void* y, int n_rows, int width, int act,

@@ -61,6 +61,19 @@ def _layer_params(block, names: dict) -> dict:
     return out
 
 
+def build_junctions(spec, dtype) -> list:
+    """The parts of the spec's junctions, in their order."""
+    return [lookup("junction", j.part.kind)(j.part, dtype) for j in spec.junctions]
+
+
+def _junction_params(part, names: dict) -> dict:
+    """``{checkpoint name: (logical name, ParamSpec)}`` of one junction."""
+    wanted = part.param_specs()
+    if set(wanted) != set(names):
+        raise ValueError(f"a junction has parameters {sorted(wanted)}; the spec names {sorted(names)}")
+    return {names[logical]: (logical, pspec) for logical, pspec in wanted.items()}
+
+
 def _final_norm_params(spec, norm=None) -> dict:
     """``{checkpoint name: (logical name, ParamSpec)}`` of the final norm."""
     if norm is None:
@@ -73,9 +86,12 @@ def _final_norm_params(spec, norm=None) -> dict:
 
 
 def expected_tensors(spec) -> dict:
-    """``{checkpoint name: ParamSpec}`` in a fixed order: embedding, layers, final norm, head."""
+    """``{checkpoint name: ParamSpec}`` in a fixed order: embedding, junctions, layers, final norm, head."""
     blocks, _ = build_layers(spec, torch.float32, "cpu")
     out = {spec.embed_name: ParamSpec((spec.vocab_size, spec.hidden_size))}
+    for part, junction in zip(build_junctions(spec, torch.float32), spec.junctions):
+        for name, (_, pspec) in _junction_params(part, junction.names).items():
+            out[name] = pspec
     for block, layer in zip(blocks, spec.layers):
         for name, (_, _, pspec) in _layer_params(block, layer.names).items():
             out[name] = pspec
@@ -115,7 +131,13 @@ class DecoderModel:
         self.depth_levels = max((b.levels for b in self.blocks), default=1) if self.depth_residual else 0
         if not self.float_residual and spec.embedding_scale != 1.0:
             raise ValueError("an embedding scale needs layers that keep a float32 residual stream")
+        self.junctions = build_junctions(spec, dtype)
+        for junction in self.junctions:
+            if kinds != {junction.residual_kind}:
+                raise ValueError(f"a junction stands in a {junction.residual_kind} residual stream; the layers keep another")
         for entry in spec.schedule:
+            if entry.junction is not None and not 0 <= entry.junction < len(self.junctions):
+                raise ValueError(f"the run order names junction {entry.junction}; the model has {len(self.junctions)}")
             if not 0 <= entry.layer < len(self.blocks):
                 raise ValueError(f"the run order names layer {entry.layer}; the model has {len(self.blocks)}")
         writers = {}
@@ -141,6 +163,9 @@ class DecoderModel:
         self.lm_head = self.embed if spec.tie_embeddings else tensors[spec.lm_head_name]
         self.final_norm.set_params({logical: tensors[name] for name, (logical, _)
                                     in _final_norm_params(spec, self.final_norm).items()})
+        for part, junction in zip(self.junctions, spec.junctions):
+            part.set_params({logical: tensors[name] for name, (logical, _)
+                             in _junction_params(part, junction.names).items()})
         for block, layer in zip(self.blocks, spec.layers):
             grouped = {}
             wanted = _layer_params(block, layer.names)
@@ -199,6 +224,9 @@ class DecoderModel:
         ctx.fenced = True
         pending = None
         for entry in self.spec.schedule:
+            if entry.junction is not None:
+                residual = self.junctions[entry.junction](residual, pending, ctx, self.embed, self.spec.embedding_scale)
+                pending = None
             residual, pending = self.blocks[entry.layer](residual, pending, ctx, entry.cache,
                                                          entry.writes_cache)
         return residual, pending
@@ -230,4 +258,6 @@ class DecoderModel:
         total = self.final_norm.weight_bytes() + self.lm_head.numel() * self.lm_head.element_size()
         for entry in self.spec.schedule:
             total += sum(p.weight_bytes() for p in self.blocks[entry.layer].parts().values())
+            if entry.junction is not None:
+                total += self.junctions[entry.junction].weight_bytes()
         return total

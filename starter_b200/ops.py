@@ -1331,21 +1331,24 @@ def residual_norm(x, dtype, eps, pending=None, next_gain=None, rows=None):
     """One kernel between two sublayers of a model whose residual stream ``x`` is float32 ``[T, H]`` and
     whose sublayers have a norm behind them as well as in front.
 
-    ``pending = (y, post_gain, bias, post_eps)``: the output ``y`` ``[T, H]`` (in ``dtype``) of the sublayer
+    ``pending = (y, post_gain, bias, post_eps[, second])``: the output ``y`` ``[T, H]`` (in ``dtype``) of the sublayer
     before, with a float32 ``bias`` ``[H]`` still to be added to it (or None); it is RMS-normed with
-    ``post_gain`` (float32 ``[H]``; None: taken as it is) and ``post_eps`` and added onto ``x`` in place.  ``next_gain``
+    ``post_gain`` (float32 ``[H]``; None: taken as it is) and ``post_eps`` and added onto ``x`` in place, and so is ``second``
+    as it is (``[T, H]`` in ``dtype``, or None: the output of a sublayer that ran beside it).  ``next_gain``
     (float32 ``[H]``): the RMS norm of the new row is returned in ``dtype``; None: nothing is returned.
     With ``rows`` (int32 ``[R]``) only those rows are computed, ``x`` is left as it was and the result is
     ``[R, H]``.  Sums, norms and the row itself are float32; the gains are the factors themselves."""
     _need(x, "x", torch.float32, 2)
     n_tokens, hidden = x.shape
-    y = post = bias = None
+    y = y2 = post = bias = None
     post_eps = eps
     if pending is not None:
-        y, post, bias, post_eps = pending
-        _need(y, "y", dtype, 2)
-        if tuple(y.shape) != (n_tokens, hidden):
-            raise KernelError(f"y {tuple(y.shape)} does not match the residual stream {tuple(x.shape)}")
+        y, post, bias, post_eps = pending[:4]
+        y2 = pending[4] if len(pending) > 4 else None
+        for t in (y,) if y2 is None else (y, y2):
+            _need(t, "y", dtype, 2)
+            if tuple(t.shape) != (n_tokens, hidden):
+                raise KernelError(f"y {tuple(t.shape)} does not match the residual stream {tuple(x.shape)}")
         if post is not None:
             _f32(post, "post gain", (hidden,))
         if bias is not None:
@@ -1359,9 +1362,35 @@ def residual_norm(x, dtype, eps, pending=None, next_gain=None, rows=None):
         _f32(next_gain, "next gain", (hidden,))
         out = torch.empty((n_rows, hidden), dtype=dtype, device=x.device)
     rc = _lib("residual32").sb_residual_norm(
-        _code(dtype), _ptr(x), _ptr(y), _ptr(bias), _ptr(post), _ptr(next_gain), _ptr(out), _ptr(rows), n_rows,
+        _code(dtype), _ptr(x), _ptr(y), _ptr(y2), _ptr(bias), _ptr(post), _ptr(next_gain), _ptr(out), _ptr(rows), n_rows,
         hidden, ctypes.c_float(post_eps), ctypes.c_float(eps), _stream())
     _check(rc, "residual_norm")
+    return out
+
+
+def residual_join(x, pending, tokens, table, scale=1.0):
+    """``[x + pending | table[tokens] * scale]`` in the type of ``table``, ``[T, 2 * H]``, for a float32 residual stream ``x``
+    ``[T, H]``; ``pending`` None or as ``residual_norm`` takes it, without a norm and a bias.  ``x`` is left as it was."""
+    _need(x, "x", torch.float32, 2)
+    n_tokens, hidden = x.shape
+    _need(tokens, "tokens", torch.int32, 1)
+    _need(table, "table", None, 2)
+    if tokens.shape[0] != n_tokens or table.shape[1] != hidden:
+        raise KernelError(f"{tuple(tokens.shape)} tokens and a table {tuple(table.shape)} do not fit the stream {tuple(x.shape)}")
+    y = y2 = None
+    if pending is not None:
+        y, y2 = pending[0], pending[4] if len(pending) > 4 else None
+        if pending[1] is not None or pending[2] is not None:
+            raise KernelError("a sublayer's output with a norm or a bias behind it cannot be joined with the embedding")
+        for t in (y,) if y2 is None else (y, y2):
+            _need(t, "y", table.dtype, 2)
+            if tuple(t.shape) != (n_tokens, hidden):
+                raise KernelError(f"y {tuple(t.shape)} does not match the residual stream {tuple(x.shape)}")
+    out = torch.empty((n_tokens, 2 * hidden), dtype=table.dtype, device=x.device)
+    rc = _lib("residual32").sb_residual_join(
+        _code(table.dtype), _ptr(x), _ptr(y), _ptr(y2), _ptr(tokens), _ptr(table), _ptr(out), n_tokens, hidden,
+        table.shape[0], ctypes.c_float(scale), _stream())
+    _check(rc, "residual_join")
     return out
 
 
@@ -1478,15 +1507,17 @@ def latent_tables(rotation, rot_dims: int):
 
 
 def latent_prepare(proj, q_gain, kv_gain, eps, cos_table, sin_table, tok_pos, tok_slot, block_table, store,
-                   q_rank, rank, rot, rot_dims, write_cache=True, layout="interleaved"):
-    """What follows a token's stacked down-projections ``proj`` = ``[query latent | key/value latent | shared
-    key part]`` (the query latent alone with ``write_cache`` false): returns the RMS-normed query latent
+                   q_rank, rank, rot, rot_dims, write_cache=True, layout="interleaved", kv_col=None):
+    """What follows a token's stacked down-projections ``proj`` = ``[query latent | .. | key/value latent | shared
+    key part]``, the key/value latent from column ``kv_col`` on (None: right behind the query latent; with ``write_cache``
+    false the row ends in front of it): returns the RMS-normed query latent
     ``[T, q_rank]``; norms the key/value latent, turns the shared key part by the token's position and files
     both in the token's row of ``store`` ``[pages, 1, 64, rank + rot]``."""
     _need(proj, "proj", None, 2)
     n_tokens = proj.shape[0]
-    want = q_rank + (rank + rot if write_cache else 0)
-    if proj.shape[1] != want:
+    kv_col = q_rank if kv_col is None else kv_col
+    want = kv_col + (rank + rot if write_cache else 0)
+    if proj.shape[1] != want or kv_col < q_rank:
         raise KernelError(f"proj has width {proj.shape[1]}, expected {want}")
     _f32(q_gain, "query latent gain", (q_rank,))
     _f32(cos_table, "cos_table")
@@ -1506,7 +1537,7 @@ def latent_prepare(proj, q_gain, kv_gain, eps, cos_table, sin_table, tok_pos, to
         _code(proj.dtype), _ptr(proj), proj.shape[1], _ptr(q_gain), _ptr(kv_gain if write_cache else None),
         ctypes.c_float(eps), _ptr(cos_table), _ptr(sin_table), cos_table.shape[1], _ptr(tok_pos), _ptr(tok_slot),
         _ptr(block_table), block_table.shape[1], _ptr(store if write_cache else None), _ptr(cq), n_tokens, q_rank,
-        rank, rot, rot_dims, int(write_cache), LATENT_LAYOUTS[layout], _stream())
+        kv_col, rank, rot, rot_dims, int(write_cache), LATENT_LAYOUTS[layout], _stream())
     _check(rc, "latent_prepare")
     return cq
 
@@ -1524,10 +1555,16 @@ def latent_rotate_q(q, qa, cos_table, sin_table, tok_pos, heads, dim, rot, rot_d
     _check(rc, "latent_rotate_q")
 
 
-def latent_attention(qa, store, block_table, tok_slot, tok_pos, heads, rank, rot, scale, window=None):
+def _latent_sink(sink, heads):
+    if sink is not None:
+        _f32(sink, "sink", (heads,))
+    return _ptr(sink)
+
+
+def latent_attention(qa, store, block_table, tok_slot, tok_pos, heads, rank, rot, scale, window=None, sink=None):
     """Softmax attention of every query row over its sequence's cached latent rows: ``qa`` ``[T, heads, rank
     + rot]`` (queries with the key up-projection folded in, then the rotated part), ``store`` ``[pages, 1,
-    64, rank + rot]``; returns ``[T, heads, rank]``, the weighted sums of the latents."""
+    64, rank + rot]``; ``sink`` (float32 ``[heads]`` or None): one more term ``exp(sink_h)`` in the denominator; returns ``[T, heads, rank]``, the weighted sums of the latents."""
     _need(qa, "qa", None, 3)
     n_tokens = qa.shape[0]
     if tuple(qa.shape[1:]) != (heads, rank + rot):
@@ -1543,7 +1580,7 @@ def latent_attention(qa, store, block_table, tok_slot, tok_pos, heads, rank, rot
     out = torch.empty((n_tokens, heads, rank), dtype=qa.dtype, device=qa.device)
     rc = _lib("attention_latent").sb_latent_attention(
         _code(qa.dtype), _ptr(qa), _ptr(out), _ptr(store), _ptr(block_table), block_table.shape[1], _ptr(tok_slot),
-        _ptr(tok_pos), n_tokens, heads, rank, rot, ctypes.c_float(scale), int(window or 0), _stream())
+        _ptr(tok_pos), n_tokens, heads, rank, rot, ctypes.c_float(scale), int(window or 0), _latent_sink(sink, heads), _stream())
     _check(rc, "latent_attention")
     return out
 
@@ -1555,7 +1592,7 @@ def latent_tc_takes(dtype, rank: int, rot: int) -> bool:
 
 
 def latent_attention_tc(qa, store, block_table, seq_slot, seq_q_start, seq_q_len, seq_kv_len, tile_seq, tile_first,
-                        heads, rank, rot, scale, window=None, n_splits=1, max_q_len=0):
+                        heads, rank, rot, scale, window=None, n_splits=1, max_q_len=0, sink=None):
     """``latent_attention`` on tensor cores (bfloat16): a block takes the heads of consecutive tokens of a
     sequence (up to 64 query rows), which all score the same cache rows.  The ``seq_*`` arrays describe the
     sequences of the step, ``tile_seq`` / ``tile_first`` list its tiles of 64 tokens.  ``n_splits`` > 1 deals
@@ -1585,7 +1622,7 @@ def latent_attention_tc(qa, store, block_table, seq_slot, seq_q_start, seq_q_len
         _ptr(qa), _ptr(out), _ptr(part_acc), _ptr(part_ml), _ptr(store), _ptr(block_table), block_table.shape[1],
         _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), _ptr(seq_kv_len), _ptr(tile_seq), _ptr(tile_first),
         tile_seq.shape[0], n_tokens, heads, rank, rot, ctypes.c_float(scale), int(window or 0), n_splits,
-        int(max_q_len), _stream())
+        int(max_q_len), _latent_sink(sink, heads), _stream())
     _check(rc, "latent_attention_tc", 2 if n_splits > 1 else 1)
     return out
 
@@ -1598,15 +1635,26 @@ def latent_splits(rows: int, heads: int, window, kv_hint: int) -> int:
     return max(1, min(32, 148 // max(1, blocks), -(-max(keys, 1) // 32)))
 
 
-def latent_attention_step(qa, store, block_table, ctx, heads, rank, rot, scale, window=None):
+def latent_attention_step(qa, store, block_table, ctx, heads, rank, rot, scale, window=None, sink=None):
     """``latent_attention`` for the step ``ctx`` describes, on the kernel that fits its shape: tensor cores
     for bfloat16 at sizes they take, the plain kernel otherwise (float32, other sizes)."""
     if latent_tc_takes(qa.dtype, rank, rot):
         splits = latent_splits(ctx.n_seqs, heads, window, ctx.max_kv_len) if ctx.max_q_len == 1 else 1
         return latent_attention_tc(qa, store, block_table, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len,
                                    ctx.seq_kv_len, ctx.tile_seq, ctx.tile_first, heads, rank, rot, scale, window,
-                                   splits, ctx.max_q_len)
-    return latent_attention(qa, store, block_table, ctx.tok_slot, ctx.tok_pos, heads, rank, rot, scale, window)
+                                   splits, ctx.max_q_len, sink)
+    return latent_attention(qa, store, block_table, ctx.tok_slot, ctx.tok_pos, heads, rank, rot, scale, window, sink)
+
+
+def sigmoid_gate(a, gate, gate_col):
+    """``a *= sigmoid(gate)`` in place for ``a`` ``[T, N]`` and the columns ``gate_col .. gate_col + N`` of ``gate`` ``[T, M]``."""
+    _need(a, "a", None, 2)
+    _need(gate, "gate", a.dtype, 2)
+    if gate.shape[0] != a.shape[0] or gate_col < 0 or gate_col + a.shape[1] > gate.shape[1]:
+        raise KernelError(f"{a.shape[1]} columns from {gate_col} of {tuple(gate.shape)} do not gate {tuple(a.shape)}")
+    rc = _lib("elementwise").sb_sigmoid_gate(_code(a.dtype), _ptr(a), _at(gate, gate_col), gate.shape[1], a.shape[1],
+                                             a.shape[0], _stream())
+    _check(rc, "sigmoid_gate")
 
 
 # ---------------------------------------------------------------------------------------- routed experts
@@ -1923,12 +1971,13 @@ def sink_prepare_rot(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block_
     _check(rc, "sink_prepare_rot")
 
 
-def sink_prepare_half(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block_table, k_store, v_store, rotation=None,
+def sink_prepare_norm(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block_table, k_store, v_store, rotation=None,
                       row_norm=None, unit_values=False, eps=0.0, write_cache=True):
-    """``sink_prepare_rot`` for half-split rotations, with norms: ``proj`` = ``[q | k | v]`` (``[q]`` with ``write_cache``
+    """``sink_prepare_rot`` for rotations of either layout, with norms: ``proj`` = ``[q | k | v]`` (``[q]`` with ``write_cache``
     false; up to 7 unused entries may follow).  ``row_norm = (q_gain, k_gain)`` (float32 ``[heads * dim]``, ``[kv_heads *
     dim]`` or None when nothing is filed): queries and keys are RMS-normed over their whole rows first.  ``rotation`` (a
-    half-split ``Rotation`` or None): entry ``i`` of its leading dimensions turns with entry ``i + dims / 2``.
+    ``Rotation`` or None): entry ``i`` of a head's leading ``dims`` entries turns with entry ``i + dims / 2`` (half-split
+    layout), or entry ``2i`` with entry ``2i + 1`` (interleaved).
     ``unit_values``: a head's value is RMS-normed without a gain.  Queries change in place, keys and values are
     filed in the cache; ``eps`` stands inside every root."""
     _need(proj, "proj", None, 2)
@@ -1939,12 +1988,13 @@ def sink_prepare_half(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block
     _need(tok_pos, "tok_pos", torch.int32, 1)
     _need(tok_slot, "tok_slot", torch.int32, 1)
     _need(block_table, "block_table", torch.int32, 2)
-    rot, cos_table, sin_table = 0, None, None
+    rot, cos_table, sin_table, pairs = 0, None, None, 0
     if rotation is not None:
         rot, cos_table, sin_table = rotation.rotary_dim, rotation.cos, rotation.sin
-        if rotation.layout != "half_split" or rot > dim or rot % 2:
-            raise KernelError(f"this kernel turns up to {dim} leading entries of a head in half-split layout; asked for {rot} "
-                              f"in {rotation.layout!r} layout")
+        pairs = int(rotation.layout == "interleaved")
+        if rotation.layout not in ("half_split", "interleaved") or rot > dim or rot % 2:
+            raise KernelError(f"this kernel turns up to {dim} leading entries of a head in half-split or interleaved layout; "
+                              f"asked for {rot} in {rotation.layout!r} layout")
         _need(cos_table, "cos table", torch.float32, 2)
         _need(sin_table, "sin table", torch.float32, 2)
         if cos_table.shape[1] != rot // 2 or tuple(sin_table.shape) != tuple(cos_table.shape):
@@ -1961,12 +2011,12 @@ def sink_prepare_half(proj, heads, kv_heads, dim, vdim, tok_pos, tok_slot, block
         if tuple(k_store.shape[1:]) != (kv_heads, PAGE_TOKENS, dim) or tuple(v_store.shape[1:]) != (kv_heads, PAGE_TOKENS, vdim):
             raise KernelError(f"cache pages have shapes {tuple(k_store.shape)} / {tuple(v_store.shape)}, expected "
                               f"[pages, {kv_heads}, {PAGE_TOKENS}, {dim}] / [.., {vdim}]")
-    rc = _lib("attention_sink").sb_sink_prepare_half(
+    rc = _lib("attention_sink").sb_sink_prepare_norm(
         _code(proj.dtype), _ptr(proj), proj.shape[1], _ptr(tok_pos), _ptr(tok_slot), _ptr(block_table),
         block_table.shape[1], _ptr(k_store if write_cache else None), _ptr(v_store if write_cache else None),
         _ptr(cos_table), _ptr(sin_table), rot, _ptr(q_gain), _ptr(k_gain), ctypes.c_float(eps), int(unit_values), n_tokens,
-        heads, kv_heads, dim, vdim, int(write_cache), _stream())
-    _check(rc, "sink_prepare_half")
+        heads, kv_heads, dim, vdim, int(write_cache), pairs, _stream())
+    _check(rc, "sink_prepare_norm")
 
 
 def _sink_check(q, k_store, v_store, heads, kv_heads, dim, vdim, penalty, sink, gate):
@@ -2253,7 +2303,7 @@ def glru_scan(u, gates, r_bias, i_bias, lam, decay_scale, proj, y_col, y_bias, s
 
 # ---------------------------------------------------------------------------------------- recurrences with a matrix state
 
-SCAN_MODES = {"state_space": 0, "gated_delta": 1, "forget_write": 2}
+SCAN_MODES = {"state_space": 0, "gated_delta": 1, "forget_write": 2, "channel_decay": 3}
 
 
 def scan_max_state() -> int:
@@ -2261,7 +2311,7 @@ def scan_max_state() -> int:
 
 
 def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_at, seq_slot, seq_q_start, seq_q_len,
-               heads, groups, n_state, v_dim):
+               heads, groups, n_state, v_dim, decay=None):
     """A linear recurrence with a state ``S`` ``[n_state, v_dim]`` per head over the sequences of a step.
 
     ``q, k, v, a_raw, b_raw`` are ``(tensor [T, N], first column)`` pairs of the working type: ``groups`` heads of
@@ -2274,7 +2324,9 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
     <- S + k u^T``, ``o = S^T q``.  ``"forget_write"`` (``groups`` = ``heads``; ``a_raw``, ``b_raw`` None): ``q <- silu(q)``,
     ``k`` holds the logits of a forget gate ``f = A_log + (1 - A_log) sigmoid(k + dt_bias)`` per row of the state, with
     lower bounds in ``A_log`` and biases in ``dt_bias`` (float32 ``[heads * n_state]`` each); ``S <- diag(f) S + (1 - f)
-    v^T``, ``o = S^T q``.  ``state`` float32 ``[slots, M]``: a slot's ``[heads, n_state, v_dim]`` from
+    v^T``, ``o = S^T q``.  ``"channel_decay"`` (``groups`` = ``heads``; ``a_raw``, ``b_raw``, ``A_log``, ``dt_bias`` None): ``decay``
+    float32 ``[T, heads * n_state]`` holds the decays' complements ``d = 1 - alpha`` per row of the state; q times ``n_state **
+    -0.5``; ``S <- diag(1 - d) S + k v^T``, ``o = S^T q``.  ``state`` float32 ``[slots, M]``: a slot's ``[heads, n_state, v_dim]`` from
     ``state_at`` on, read at the start and written at the end.  Returns float32 ``[T, heads * v_dim]``."""
     if mode not in SCAN_MODES:
         raise KernelError(f"no recurrence {mode!r} (known: {', '.join(SCAN_MODES)})")
@@ -2291,9 +2343,14 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
         if t.shape[0] != n_tokens or col < 0 or col + width > t.shape[1]:
             raise KernelError(f"{name}: {width} columns from {col} of {tuple(t.shape)} do not fit {n_tokens} tokens")
         args += [_at(t, col), t.shape[1]]
-    per_head = heads * n_state if mode == "forget_write" else heads
-    _f32(A_log, "A_log", (per_head,))
-    _f32(dt_bias, "dt_bias", (per_head,))
+    if (mode == "channel_decay") != (decay is not None):
+        raise KernelError("decays per row of the state belong to the channel_decay recurrence")
+    if decay is not None:
+        _f32(decay, "decay", (n_tokens, heads * n_state))
+    else:
+        per_head = heads * n_state if mode == "forget_write" else heads
+        _f32(A_log, "A_log", (per_head,))
+        _f32(dt_bias, "dt_bias", (per_head,))
     if skip is not None:
         _f32(skip, "skip", (heads,))
     _need(state, "state", torch.float32, 2)
@@ -2302,13 +2359,34 @@ def state_scan(mode, q, k, v, a_raw, b_raw, A_log, dt_bias, skip, state, state_a
     n_seqs = _seq_arrays(seq_slot, seq_q_start, seq_q_len)
     out = torch.empty((n_tokens, heads * v_dim), dtype=torch.float32, device=state.device)
     rc = _lib("state_scan").sb_state_scan(
-        _code(dtype), SCAN_MODES[mode], *args, _ptr(A_log), _ptr(dt_bias), _ptr(skip), _at(state, state_at),
+        _code(dtype), SCAN_MODES[mode], *args, _ptr(A_log), _ptr(dt_bias), _ptr(skip), _ptr(decay), _at(state, state_at),
         ctypes.c_longlong(state.shape[1]), _ptr(out), _ptr(seq_slot), _ptr(seq_q_start), _ptr(seq_q_len), n_seqs, heads,
         groups, n_state, v_dim, _stream())
     if rc == -2:
         raise KernelError(f"the recurrence takes states of 1 to {scan_max_state()} rows and heads in whole groups, not "
                           f"{n_state} rows, {heads} heads, {groups} groups")
     _check(rc, "state_scan")
+    return out
+
+
+def low_rank_decay(u, col, a2, bias, tau):
+    """``1 - sigmoid(z) ** (1 / tau)`` with ``z = u @ a2 + bias``: how much of its row of a recurrent state every channel lets
+    go of a token.  ``u``: the columns ``col .. col + R`` of a ``[T, N]`` tensor; ``a2`` float32 ``[R, C]``, ``bias`` float32
+    ``[C]``.  The product, the logarithm and the exponential are float; returns float32 ``[T, C]``."""
+    _need(u, "u", None, 2)
+    _need(a2, "a2", torch.float32, 2)
+    rank, channels = a2.shape
+    _f32(bias, "bias", (channels,))
+    if col < 0 or col + rank > u.shape[1]:
+        raise KernelError(f"{rank} columns from {col} of {tuple(u.shape)} are not there")
+    if not tau > 0.0:
+        raise KernelError(f"tau={tau} must be positive")
+    out = torch.empty((u.shape[0], channels), dtype=torch.float32, device=u.device)
+    rc = _lib("state_scan").sb_low_rank_decay(_code(u.dtype), _at(u, col), u.shape[1], _ptr(a2), _ptr(bias), _ptr(out),
+                                              u.shape[0], channels, rank, ctypes.c_float(1.0 / tau), _stream())
+    if rc == -2:
+        raise KernelError(f"the low-rank decay takes ranks of 1 to 1024, not {rank}")
+    _check(rc, "low_rank_decay")
     return out
 
 

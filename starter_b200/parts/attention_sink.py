@@ -31,14 +31,13 @@ class SinkAttention(Part):
             raise ValueError("the attention's spec and the position part it is handed do not agree")
         if spec.window is None and spec.chunk is None and spec.keep_first:
             raise ValueError("first keys are kept by a window or a chunk; this attention sees all keys")
-        #: which kernel follows the projections: the half-split rotation with norms, the interleaved one, or none
-        self.half_split = (getattr(spec.position, "kind", None) == "rope_partial" or spec.row_norm or spec.unit_values)
-        if self.half_split and getattr(spec.position, "kind", "rope_partial") != "rope_partial":
-            raise ValueError("norms of queries, keys and values go with half-split rotary positions")
-        if (position is not None or spec.values_from_keys or self.half_split) and spec.head_gate:
+        #: which kernel follows the projections: the one with norms (either rotation; the half-split one always), the
+        #: one with the interleaved rotation alone, or the one without a rotation
+        self.normed = getattr(spec.position, "kind", None) == "rope_partial" or spec.row_norm or spec.unit_values
+        if (position is not None or spec.values_from_keys or self.normed) and spec.head_gate:
             raise ValueError("head gates are formed by the kernel that files keys and values without a rotation")
-        if self.half_split and spec.values_from_keys:
-            raise ValueError("values taken from the keys go with interleaved rotary positions")
+        if self.normed and spec.values_from_keys:
+            raise ValueError("values taken from the keys go with interleaved rotary positions and no norms")
         if (spec.conv is not None or spec.bias) and spec.head_gate:
             raise ValueError("head gates have no bias and no convolution")
         if not spec.own_kv and (spec.conv is not None or spec.bias or spec.values_from_keys):
@@ -169,9 +168,9 @@ class SinkAttention(Part):
         if self.taps is not None:
             proj = ops.short_conv(proj, 0, self.convolved, self.taps, None, self.biases, cache.entry_state(entry),
                                   self.state_at, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len, ctx.max_q_len)
-        if self.half_split:
+        if self.normed:
             # queries normed and turned in place; keys normed and turned, values normed on their way into the cache
-            ops.sink_prepare_half(proj, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, ctx.tok_pos, ctx.tok_slot,
+            ops.sink_prepare_norm(proj, s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim, ctx.tok_pos, ctx.tok_slot,
                                   cache.block_table, keys, values,
                                   self.position.rotation() if self.position is not None else None, self.row_norm,
                                   s.unit_values, s.norm_eps, write_cache=writes_cache)

@@ -50,13 +50,15 @@ class PreNormBlock:
 
 @dataclass
 class Summand:
-    """A sublayer's output not yet added onto a float32 residual stream (it is added as it is)."""
+    """A sublayer's output not yet added onto a float32 residual stream (it is added as it is); ``second``: the output
+    of a sublayer that ran beside it, to be added too."""
 
     value: object
     eps: float = 0.0
+    second: object = None
 
     def for_kernel(self):
-        return self.value, None, None, self.eps
+        return self.value, None, None, self.eps, self.second
 
 
 class PreNorm32Block:
@@ -100,3 +102,15 @@ class PreNorm32MixerOnlyBlock(PreNorm32Block):
     """The same layer without a feed-forward (and so without the second norm)."""
 
     FAMILIES = {"mixer": "mixer", "norm1": "norm"}
+
+
+class ParallelPreNorm32Block(PreNorm32Block):
+    """Both sublayers read the same norm and are added together: ``x <- x + (mixer(norm1(x)) + feed_forward(norm1(x)))``
+    around a residual stream that is a 32-bit sum.  The two outputs stay open until the next layer's norm (or whatever
+    comes next) adds both in one kernel."""
+
+    FAMILIES = {"mixer": "mixer", "feed_forward": "feed_forward", "norm1": "norm"}
+
+    def __call__(self, residual, pending, ctx, entry, writes_cache=True):
+        n = self._open(residual, pending, self.norm1)
+        return residual, Summand(self.mixer(n, ctx, entry, writes_cache), second=self.feed_forward(n, ctx))

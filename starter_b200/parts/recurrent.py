@@ -8,7 +8,9 @@ whose last inputs are part of that state:
 * ``GatedDeltaMixer``: the gated delta rule on unit queries and keys (the same three kernels, the scan in its
   ``gated_delta`` form);
 * ``ForgetWriteMixer``: one gate per key channel for what is kept and what is written (no convolution; the scan in
-  its ``forget_write`` form, ``ops.group_norm_gate`` without a gate).
+  its ``forget_write`` form, ``ops.group_norm_gate`` without a gate);
+* ``GatedLinearAttention``: keys written as they are over rows that decay per key channel (no convolution;
+  ``ops.low_rank_decay`` forms the decays, the scan in its ``channel_decay`` form, ``ops.group_norm_gate``).
 
 A whole prompt, a later portion and a single token are the same code, and a step captured in a CUDA graph too:
 the kernels work from the step's device arrays and the slots.  A slot's floats: the convolution's last ``taps -
@@ -247,3 +249,50 @@ class ForgetWriteMixer(_Recurrent):
 
     def weight_bytes(self):
         return bytes_of(self.stacked, self.f_bias, self.lower, self.gain, self.o)
+
+
+class GatedLinearAttention(_Recurrent):
+    def __init__(self, spec, dtype, position=None):
+        super().__init__(spec, dtype, position)
+        if not spec.tau > 0.0:
+            raise ValueError(f"a decay's root needs a positive tau, not {spec.tau}")
+        self.qk = spec.num_heads * spec.head_dim
+        self.inner = spec.num_heads * spec.value_dim
+
+    def state_need(self):
+        s = self.spec
+        return StateNeed((s.num_heads * s.head_dim * s.value_dim,), "float32")
+
+    def param_specs(self):
+        s = self.spec
+        return {
+            "q": ParamSpec((self.qk, s.hidden_size)), "k": ParamSpec((self.qk, s.hidden_size)),
+            "v": ParamSpec((self.inner, s.hidden_size)), "g": ParamSpec((self.inner, s.hidden_size)),
+            "a1": ParamSpec((s.decay_rank, s.hidden_size)), "a2": ParamSpec((self.qk, s.decay_rank), "matrix32"),
+            "a2_bias": ParamSpec((self.qk,), "bias32"), "norm": ParamSpec((s.value_dim,), "gain32"),
+            "o": ParamSpec((s.hidden_size, self.inner)),
+        }
+
+    def set_params(self, params):
+        # one product for [q | k | v | g | a1]
+        self.stacked = _padded_rows([params[n] for n in ("q", "k", "v", "g", "a1")], self.spec.hidden_size)
+        # (transposed: the channels of one rank entry lie side by side)
+        self.a2 = params["a2"].float().t().contiguous()
+        self.a2_bias = params["a2_bias"].float().contiguous()
+        self.gain = params["norm"].float().contiguous()
+        self.o = params["o"].contiguous()
+
+    def __call__(self, x, ctx, entry, writes_cache=True):
+        s = self.spec
+        state = self._state(ctx, entry, writes_cache)
+        gate_at = 2 * self.qk + self.inner
+        proj = ops.linear(x, self.stacked, status=ctx.status)
+        decay = ops.low_rank_decay(proj, gate_at + self.inner, self.a2, self.a2_bias, s.tau)
+        o = ops.state_scan("channel_decay", (proj, 0), (proj, self.qk), (proj, 2 * self.qk), None, None, None, None, None,
+                           state, self.state_at, ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len, s.num_heads, s.num_heads,
+                           s.head_dim, s.value_dim, decay=decay)
+        y = ops.group_norm_gate(o, proj, gate_at, self.gain, s.num_heads, s.norm_eps, False, x.dtype)
+        return ops.linear(y, self.o, status=ctx.status)
+
+    def weight_bytes(self):
+        return bytes_of(self.stacked, self.a2, self.a2_bias, self.gain, self.o)

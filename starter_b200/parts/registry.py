@@ -19,6 +19,8 @@ Families and their interfaces
   arrangement   class attribute ``FAMILIES`` (part name -> family); ``__init__(parts: dict)``;
                 ``parts()``; attribute ``mixer`` (the part that owns the layer's cache entry);
                 ``__call__(residual, pending, ctx, entry, writes_cache)`` -> ``(residual, pending)``
+  junction      ``__init__(spec, dtype)``; ``param_specs()``, ``set_params``; attribute ``residual_kind`` (the streams it
+                stands in); ``__call__(residual, pending, ctx, table, scale)`` -> the new residual stream, nothing pending
 """
 
 from __future__ import annotations
@@ -27,20 +29,21 @@ from .attention import GroupedQueryAttention
 from .attention_diff import DifferentialAttention
 from .attention_latent import LatentAttention
 from .attention_sink import SinkAttention
-from .block import PreNorm32Block, PreNorm32MixerOnlyBlock, PreNormBlock
+from .block import ParallelPreNorm32Block, PreNorm32Block, PreNorm32MixerOnlyBlock, PreNormBlock
 from .depth import DepthAverage, DepthMixerOnlyBlock, DepthPreNormBlock
 from .feedforward import BiasedFeedForward, ClampedGatedFeedForward, GatedFeedForward, RoutedExperts
 from .hyper import HyperConnection, HyperMixerOnlyBlock, HyperPreNormBlock
+from .junction import EmbeddingJoin
 from .norm import RMSNorm
 from .parallel import ParallelMixer
-from .recurrent import ForgetWriteMixer, GatedDeltaMixer, GatedLinearRecurrence, StateSpaceMixer
+from .recurrent import ForgetWriteMixer, GatedDeltaMixer, GatedLinearAttention, GatedLinearRecurrence, StateSpaceMixer
 from .norm_dyt import DynamicTanh
 from .norm_layer import LayerNorm
 from .rotary import InterleavedRotaryTable, PartialRotaryTable, RotaryTable
 from .sandwich import SandwichBlock, SandwichMixerOnlyBlock
 from .wkv import WkvMixer
 
-FAMILIES = ("mixer", "feed_forward", "norm", "position", "connection", "arrangement")
+FAMILIES = ("mixer", "feed_forward", "norm", "position", "connection", "arrangement", "junction")
 _REGISTRY = {family: {} for family in FAMILIES}
 
 
@@ -89,3 +92,6 @@ register("mixer", "state_space", StateSpaceMixer)
 register("mixer", "gated_delta", GatedDeltaMixer)
 register("mixer", "forget_write", ForgetWriteMixer)
 register("mixer", "parallel", ParallelMixer)
+register("mixer", "gated_linear_attention", GatedLinearAttention)
+register("arrangement", "parallel32", ParallelPreNorm32Block)
+register("junction", "embedding_join", EmbeddingJoin)

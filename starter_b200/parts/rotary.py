@@ -70,17 +70,33 @@ class RotaryTable(Part):
 
 class InterleavedRotaryTable(RotaryTable):
     """Tables for a rotation of entry ``2i`` with entry ``2i + 1`` over the first ``dims`` entries of a
-    vector: ``[positions, dims / 2]`` of ``cos`` and ``sin`` of ``position * base ** (-2i / dims)``.  The
-    angles are formed in float64 on the host and the tables rounded to float32 once."""
+    vector: ``[positions, dims / 2]`` of ``cos`` and ``sin`` of ``position * base ** (-2i / dims)``.  The spec's ``scaling``
+    changes the frequencies (and, for YaRN, multiplies cos and sin).  The angles are formed in float64 on the host and
+    the tables rounded to float32 once."""
+
+    LAYOUT = "interleaved"
 
     def rotation(self) -> Rotation:
-        return Rotation(self.cos, self.sin, self.spec.dims, "interleaved")
+        return Rotation(self.cos, self.sin, self.spec.dims, self.LAYOUT)
 
     def frequencies(self):
         """``(float64 [dims / 2], multiplier of cos and sin)``."""
-        dims = self.spec.dims
+        dims, base, scaling = self.spec.dims, float(self.spec.base), self.spec.scaling
         i = torch.arange(dims // 2, dtype=torch.float64)
-        return torch.pow(torch.tensor(float(self.spec.base), dtype=torch.float64), -2.0 * i / dims), 1.0
+        freq = torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * i / dims)
+        if scaling is None:
+            return freq, 1.0
+        if not hasattr(scaling, "original"):
+            return freq / scaling.factor, 1.0
+
+        def index_of(turns: float) -> float:
+            # the (fractional) frequency that makes that many turns over the original length
+            return dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+        lo = max(math.floor(index_of(scaling.fast)), 0)
+        hi = min(math.ceil(index_of(scaling.slow)), dims - 1)
+        stretched = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        return freq / scaling.factor * stretched + freq * (1.0 - stretched), 0.1 * math.log(scaling.factor) + 1.0
 
     def ensure(self, length: int) -> bool:
         if length <= self.length:
@@ -98,27 +114,6 @@ class InterleavedRotaryTable(RotaryTable):
 
 class PartialRotaryTable(InterleavedRotaryTable):
     """Tables for a rotation of entry ``i`` with entry ``i + dims / 2`` over the first ``dims`` entries of a
-    vector: the same angles ``position * base ** (-2i / dims)`` as the interleaved tables, paired half-split.  The
-    spec's ``scaling`` changes the frequencies (and, for YaRN, multiplies cos and sin)."""
+    vector: the same angles as the interleaved tables, paired half-split."""
 
-    def frequencies(self):
-        freq, mult = super().frequencies()
-        scaling = self.spec.scaling
-        if scaling is None:
-            return freq, mult
-        if not hasattr(scaling, "original"):
-            return freq / scaling.factor, mult
-        dims, base = self.spec.dims, float(self.spec.base)
-
-        def index_of(turns: float) -> float:
-            # the (fractional) frequency that makes that many turns over the original length
-            return dims * math.log(scaling.original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
-
-        lo = max(math.floor(index_of(scaling.fast)), 0)
-        hi = min(math.ceil(index_of(scaling.slow)), dims - 1)
-        i = torch.arange(dims // 2, dtype=torch.float64)
-        stretched = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
-        return freq / scaling.factor * stretched + freq * (1.0 - stretched), 0.1 * math.log(scaling.factor) + 1.0
-
-    def rotation(self) -> Rotation:
-        return Rotation(self.cos, self.sin, self.spec.dims, "half_split")
+    LAYOUT = "half_split"

@@ -186,14 +186,14 @@ def test_prepare_alone(heads, kv_heads, dim, vdim, turn, row_norm, unit, dtype):
     pos, slot = dev(place, torch.int32), ints([1] * n)
     norms = (dev(gains[0]), dev(gains[1])) if row_norm else None
     alone = proj[:, :widths[0]].contiguous()
-    ops.sink_prepare_half(proj, heads, kv_heads, dim, vdim, pos, slot, table, ks, vs, rotation, norms, unit, eps)
+    ops.sink_prepare_norm(proj, heads, kv_heads, dim, vdim, pos, slot, table, ks, vs, rotation, norms, unit, eps)
     close(proj[:, :widths[0]], q.reshape(n, -1), dtype, "queries", fp32=1e-6, bf16=8e-3)
     pages = torch.tensor([5, 2, 7, 0, 3])[place // 64]
     close(ks[pages.cuda(), :, (place % 64).cuda()], k, dtype, "keys", fp32=1e-6, bf16=8e-3)
     close(vs[pages.cuda(), :, (place % 64).cuda()], v, dtype, "values", fp32=1e-6, bf16=8e-3)
     assert float(ks[5, :, :37].abs().max()) == 0.0 and float(vs[3].abs().max()) == 0.0, "nothing else was written"
     kept = ks.clone()
-    ops.sink_prepare_half(alone, heads, kv_heads, dim, vdim, pos, slot, table, ks, vs, rotation,
+    ops.sink_prepare_norm(alone, heads, kv_heads, dim, vdim, pos, slot, table, ks, vs, rotation,
                           (norms[0], None) if row_norm else None, False, eps, write_cache=False)
     assert torch.equal(ks, kept)
     close(alone, q.reshape(n, -1), dtype, "a reading layer's queries", fp32=1e-6, bf16=8e-3)
