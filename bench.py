@@ -1009,6 +1009,133 @@ def setotar_compare(args) -> int:
                               beside=("bavedra", "Bavedra", bavedra_config, bavedra_kernels_alone))
 
 
+def salulorn_config(size: dict, layers: int) -> dict:
+    """Salulorn at ``size``: a recurrence, window attention and latent attention in turn, each beside a dense gated
+    feed-forward, the first two layers passed through twice (``layers`` runs of ``layers - 2`` stored layers).  Recurrent
+    states of 128 x 128 with decays of rank 16; attention heads of 128 with biases, three taps, the whole head rotated, a
+    window of 1,024 and a cap; latent attention with 128 plain + 64 rotated query/key entries and values of 128 a head
+    over a latent of 512, stretched by parts."""
+    w, out = size["width"], []
+    dense = dict(kind="dense", ff=size["ff"])
+    kinds = (("gla", dict(heads=w // 128, dim=128, vdim=128, tau=16.0, decay_rank=16)),
+             ("attention", dict(heads=size["heads"], kv_heads=size["kv_heads"], dim=128, vdim=128, scale=128 ** -0.5, conv=3,
+                                mask=dict(size=1024), rot=dict(base=1e6, dims=128), softcap=50.0)),
+             ("latent_attention", dict(heads=size["heads"], dim=128, rot_dim=64, vdim=128, q_rank=w * 3 // 4 // 64 * 64, kv_rank=512,
+                                       scale=192 ** -0.5, rot=dict(base=1e4, dims=64, scaling=dict(
+                                           factor=4.0, original=8192, fast=32.0, slow=1.0)))))
+    for i in range(layers - 2):
+        kind, mixer = kinds[i % 3]
+        out.append(dict(type=kind, mixer=mixer, mlp=dense))
+    return dict(architecture="Salulorn", vocab=size["vocab"], width=w, norm=dict(eps=1e-6), layers=out,
+                loop=dict(start=0, stop=2, times=2))
+
+
+def salulorn_kernels_alone(ops, out, name, rows, x, blocks, spec, cache, ctx, size, batch, context, prompt_len, rnd,
+                           in_graph, bw, tc):
+    """Salulorn's own kernels alone at ``rows`` rows, once per layer inside a CUDA graph."""
+    import torch
+
+    w, dev, bf, is_prompt = size["width"], x.device, x.dtype, rows == prompt_len
+    seqs, n_seqs = (ctx.seq_slot, ctx.seq_q_start, ctx.seq_q_len), ctx.n_seqs
+    # (a stream a call: together more than L2 holds at the prompt's size)
+    streams = [torch.randn(rows, w, device=dev) for _ in blocks]
+    y, z = rnd(rows, w), rnd(rows, w)
+    us = in_graph([lambda b=b, s=s: ops.residual_norm(s, bf, 1e-6, (y, None, None, 0.0, z), b.norm1.weight)
+                   for b, s in zip(blocks, streams)])
+    out[f"{name}: two outputs + residual sum + norm"] = bw(us, rows * w * (4 + 4 + 2 + 2 + 2))
+    table = rnd(spec.vocab_size, w)
+    us = in_graph([lambda s=s: ops.residual_join(s, (y, None, None, 0.0, z), ctx.tokens, table) for s in streams])
+    out[f"{name}: stream and embedding side by side"] = bw(us, rows * w * (4 + 2 + 2 + 2 + 4))
+    joined, weights = rnd(rows, 2 * w), [rnd(w, 2 * w) for _ in range(8)]
+    us = in_graph([lambda m=m: ops.linear(joined, m, out_float=True) for m in weights])
+    out[f"{name}: projection back to the stream"] = tc(us, rows * 4 * w * w) if is_prompt else bw(us, 4 * w * w)
+
+    def of(kind):
+        return [(b.mixer, e.cache) for b, e in zip(blocks, spec.schedule) if b.mixer.spec.kind == kind]
+
+    pairs = of("gated_linear_attention")
+    m = pairs[0][0]
+    sp = m.spec
+    proj = rnd(rows, m.stacked.shape[0])
+    gate_at = 2 * m.qk + m.inner
+    us = in_graph([lambda p=p: ops.low_rank_decay(proj, gate_at + m.inner, p.a2, p.a2_bias, sp.tau) for p, _ in pairs])
+    out[f"{name}: decays of low rank"] = bw(us, rows * (m.qk * 4 + sp.decay_rank * 2))
+    decay = ops.low_rank_decay(proj, gate_at + m.inner, m.a2, m.a2_bias, sp.tau)
+    us = in_graph([lambda p=p, e=e: ops.state_scan("channel_decay", (proj, 0), (proj, m.qk), (proj, 2 * m.qk), None, None, None, None,
+                                                    None, cache.entry_state(e), p.state_at, *seqs, sp.num_heads, sp.num_heads,
+                                                    sp.head_dim, sp.value_dim, decay=decay) for p, e in pairs])
+    d = bw(us, rows * (m.qk * 8 + m.inner * 6) + n_seqs * sp.num_heads * sp.head_dim * sp.value_dim * 4 * 2)
+    d["gflops"] = rows * sp.num_heads * sp.head_dim * sp.value_dim * 5 / us / 1e3
+    out[f"{name}: recurrence with a decay per channel (state walk)"] = d
+    o32 = torch.randn(rows, m.inner, device=dev)
+    us = in_graph([lambda p=p: ops.group_norm_gate(o32, proj, gate_at, p.gain, sp.num_heads, 1e-6, False, bf) for p, _ in pairs])
+    out[f"{name}: head norm + gate"] = bw(us, rows * m.inner * (4 + 2 + 2))
+
+    pairs = of("sink_attention")
+    a = pairs[0][0]
+    sp = a.spec
+    heads, kvh, dim, vdim = sp.num_heads, sp.num_kv_heads, sp.head_dim, sp.value_dim
+    proj = rnd(rows, a.qkvg.shape[0])
+    us = in_graph([lambda p=p, e=e: ops.short_conv(proj, 0, a.convolved, p.taps, None, p.biases, cache.entry_state(e), p.state_at,
+                                                    *seqs, ctx.max_q_len) for p, e in pairs])
+    out[f"{name}: bias + short convolution ({a.convolved} channels)"] = bw(us, rows * a.convolved * 4 + n_seqs * (sp.conv - 1) * a.convolved * 8)
+
+    def prepare(p, e):
+        k, v = cache.entry_pages(e)
+        ops.sink_prepare_norm(proj, heads, kvh, dim, vdim, ctx.tok_pos, ctx.tok_slot, cache.block_table, k, v, a.position.rotation(),
+                              p.row_norm, False, sp.norm_eps)
+
+    def attend(p, e, sink):
+        k, v = cache.entry_pages(e)
+        return ops.sink_attention_step(proj, k, v, cache.block_table, ctx, heads, kvh, dim, vdim, sp.scale, None, sink, None, None,
+                                       sp.window, 0, sp.softcap)
+
+    us = in_graph([lambda p=p, e=e: prepare(p, e) for p, e in pairs])
+    out[f"{name}: row norms, rotation, cache write"] = bw(us, rows * 2 * (2 * heads * dim + 2 * kvh * (dim + vdim)))
+    seen = lambda p: min(p + 1, sp.window)  # noqa: E731
+    for title, with_sink in (("window, cap, sink: attention", True), ("window, cap, no sink: attention", False)):
+        us = in_graph([lambda p=p, e=e: attend(p, e, p.sink if with_sink else None) for p, e in pairs])
+        out[f"{name}: {title}"] = (tc(us, heads * 2 * (dim + vdim) * sum(seen(p) for p in range(prompt_len))) if is_prompt
+                                   else bw(us, batch * seen(context) * kvh * (dim + vdim) * 2))
+
+    pairs = of("latent_attention")
+    m = pairs[0][0]
+    sp = m.spec
+    proj = rnd(rows, m.down.shape[0])
+    cos, sin = ops.latent_tables(m.position.rotation(), sp.position.dims)
+    us = in_graph([lambda p=p, e=e: ops.latent_prepare(proj, p.q_gain, p.kv_gain, 1e-6, cos, sin, ctx.tok_pos, ctx.tok_slot,
+                                                        cache.block_table, cache.entry_pages(e)[0], sp.q_rank, sp.kv_rank, sp.rot_dim,
+                                                        sp.position.dims, kv_col=m.kv_at) for p, e in pairs])
+    out[f"{name}: latent norms, rotation, cache write"] = bw(us, rows * 2 * 2 * (sp.q_rank + m.row))
+    qa = rnd(rows, sp.num_heads, m.row)
+    forms = [("latent attention, sink", None, True), ("latent attention, no sink", None, False)]
+    forms += [("latent attention, window of 1,024, no sink (Kesedra's form)", 1024, False)]
+    for title, window, with_sink in forms:
+        us = in_graph([lambda p=p, e=e: ops.latent_attention_step(qa, cache.entry_pages(e)[0], cache.block_table, ctx, sp.num_heads,
+                                                                   sp.kv_rank, sp.rot_dim, sp.scale, window, p.sink if with_sink else None)
+                       for p, e in pairs])
+        span = lambda p: min(p + 1, window or p + 1)  # noqa: E731
+        out[f"{name}: {title}"] = (tc(us, sp.num_heads * 2 * (m.row + sp.kv_rank) * sum(span(p) for p in range(prompt_len))) if is_prompt
+                                   else bw(us, batch * span(context) * m.row * 2))
+    heads_out = rnd(rows, m.gate_size)
+    us = in_graph([lambda p=p: ops.sigmoid_gate(heads_out, proj, sp.q_rank) for p, _ in pairs])
+    out[f"{name}: output gate"] = bw(us, rows * m.gate_size * 2 * 3)
+    ff = [b.feed_forward for b in blocks]
+    us = in_graph([lambda f=f: f(x, None) for f in ff])
+    inner = ff[0].spec.intermediate_size
+    out[f"{name}: feed-forward (gate, up, down)"] = tc(us, rows * 6 * inner * w) if is_prompt else bw(us, 6 * inner * w)
+
+
+def salulorn_compare(args) -> int:
+    """Beside Setotar: the closest design this library has (window attention with biases, convolutions and capped scores,
+    row norms, a recurrence with a matrix state per head, a 32-bit residual); the latent attention is also timed in the
+    form it has in Kesedra."""
+    if args.layers_given and args.layers < 5:
+        raise SystemExit("this comparison needs 5 layers or more: three kinds, two of them run twice")
+    return compare_with_qwen3(args, "salulorn", "Salulorn", salulorn_config, salulorn_kernels_alone, ["2048"],
+                              beside=("setotar", "Setotar", setotar_config, setotar_kernels_alone))
+
+
 def kesedra_compare(args) -> int:
     # the 2048 size alone by default: at 2560 with 8 layers a prompt step of this design failed to return while
     # its kernels still released their successors early; the larger sizes have not been timed since and run
@@ -1021,7 +1148,7 @@ def korurax_compare(args) -> int:
 
 
 def compare_with_qwen3(args, design_key, design_title, config_of, own_kernels, default_sizes, beside=None) -> int:
-    """``--design kesedra`` / ``korurax`` / ``bavedra`` / ``setotar``: prefill and decode throughput of that design beside Qwen3
+    """``--design kesedra`` / ``korurax`` / ``bavedra`` / ``setotar`` / ``salulorn``: prefill and decode throughput of that design beside Qwen3
     (or, with ``beside = (key, title, config_of, kernels_alone)``, beside that design: the closest model this library
     has) at equal width, dense feed-forward, vocabulary and head count, and the design's own kernels alone beside the
     other's like kernels, each against its roofline.  Every number is timed on the device with CUDA events; the
@@ -1184,8 +1311,8 @@ def main() -> int:
                              "generation range); the cache is sized for it")
     parser.add_argument("--per-stage", action="store_true",
                         help="also print where a decode step's time goes, kernel by kernel (stderr)")
-    parser.add_argument("--design", choices=["goguvik", "kesedra", "korurax", "bavedra", "setotar"], default=None,
-                        help="instead of the default run: that design beside Qwen3 (Bavedra: Kesedra; Setotar: Bavedra) at equal "
+    parser.add_argument("--design", choices=["goguvik", "kesedra", "korurax", "bavedra", "setotar", "salulorn"], default=None,
+                        help="instead of the default run: that design beside Qwen3 (Bavedra: Kesedra; Setotar: Bavedra; Salulorn: Setotar) at equal "
                              "sizes (prefill, decode, and each design's own kernels against their rooflines)")
     parser.add_argument("--design-sizes", default=None, help="comma-separated subset of " + ",".join(DESIGN_SIZES))
     args = parser.parse_args()
@@ -1199,6 +1326,8 @@ def main() -> int:
         return workload(args)
     if args.design == "korurax":
         return korurax_compare(args)
+    if args.design == "salulorn":
+        return salulorn_compare(args)
     if args.design == "setotar":
         return setotar_compare(args)
     if args.design == "bavedra":
